@@ -5,6 +5,7 @@ from .vumezen import VumezenConfig
 from .nubedra import NubedraConfig
 from .zedirax import ZediraxConfig
 from .zetalorn import ZetalornConfig
+from .bezadra import BezadraConfig
 
-__all__ = ["CallSpec", "ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "SubLayerSpec", "Qwen2Config", "VumezenConfig", "NubedraConfig", "ZediraxConfig", "ZetalornConfig",
+__all__ = ["CallSpec", "ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "SubLayerSpec", "Qwen2Config", "VumezenConfig", "NubedraConfig", "ZediraxConfig", "ZetalornConfig", "BezadraConfig",
            "config_from_dict", "known_architectures", "load_config", "register_architecture"]

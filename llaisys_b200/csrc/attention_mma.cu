@@ -92,6 +92,7 @@ struct MmaAttnParams {
     const bf16* pool_v;
     const int* pool_table;  // [B, pool_table_stride]
     int pool_table_stride;
+    float softcap;          // > 0: scaled scores pass through softcap * tanh(. / softcap)   (not with the options above)
 };
 
 // What a thread's two score rows need beyond the common scale when scores depend on the positions themselves: the
@@ -100,6 +101,7 @@ struct RowBias {
     int q0, q1;
     float sc0, sc1;
     float r1a, r2a, r1b, r2b;
+    float cap_in, cap_out;      // capped scores: cap_out * tanh(cap_in * q.k), base-2 scale
 };
 __device__ __forceinline__ float query_temperature(const MmaAttnParams& p, int pos) {
     return p.q_temp_every > 0 ? 1.f + p.q_temp_coef * logf((float)((pos + 1) / p.q_temp_every) + 1.f) : 1.f;
@@ -270,7 +272,7 @@ __device__ __forceinline__ void load_q(uint32_t (&qf)[KSTEPS][4], F q_of, int la
 // One warp: scores of its 16 rows against NT*8 keys starting at row `key0` of the tile in `stage`,
 // masking, online softmax update, and O += P V.  lo0/hi0 and lo1/hi1: visible key positions of
 // the thread's two rows (lane/4 and lane/4 + 8).
-template <int NT, bool MASKED = true, bool BIAS = false>
+template <int NT, bool MASKED = true, bool BIAS = false, bool CAP = false>
 __device__ __forceinline__ void tile_step(const uint32_t (&qf)[KSTEPS][4], float (&o)[DTILES][4], float (&m)[2],
                                           float (&l)[2], uint32_t stage, int key0, int pos0, int lo0, int hi0, int lo1,
                                           int hi1, float scale_log2, int lane, int keep = 0, const RowBias rb = RowBias{}) {
@@ -291,9 +293,13 @@ __device__ __forceinline__ void tile_step(const uint32_t (&qf)[KSTEPS][4], float
     }
     // mask and row maxima (MASKED = false: the caller knows every key of the tile is visible to every row)
     float mx0 = -INFINITY, mx1 = -INFINITY;
-    const float sc0 = BIAS ? rb.sc0 : scale_log2, sc1 = BIAS ? rb.sc1 : scale_log2;
+    const float sc0 = CAP ? 1.f : BIAS ? rb.sc0 : scale_log2, sc1 = CAP ? 1.f : BIAS ? rb.sc1 : scale_log2;
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
+        if (CAP) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[n][e] = rb.cap_out * llb_tanh_fast(s[n][e] * rb.cap_in);
+        }
         if (MASKED) {
             int kp = pos0 + key0 + n * 8 + (lane & 3) * 2;
             s[n][0] = ((kp >= lo0 || kp < keep) && kp <= hi0) ? s[n][0] * sc0 : -INFINITY;
@@ -435,7 +441,7 @@ __device__ __forceinline__ void cluster_merge(int S, int n_heads, uint32_t ml_ad
 }
 
 // ------------------------------------------------------------------ decode
-template <int NST, bool BIAS = false>
+template <int NST, bool BIAS = false, bool CAP = false>
 __global__ void __launch_bounds__(THREADS) attn_mma_decode_kernel(MmaAttnParams p) {
     extern __shared__ uint8_t smem_raw[];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -583,6 +589,10 @@ __global__ void __launch_bounds__(THREADS) attn_mma_decode_kernel(MmaAttnParams 
         rb.r1b = p.dist_r1 ? p.dist_r1[hb] : 0.f;
         rb.r2b = p.dist_r2 ? p.dist_r2[hb] : 0.f;
     }
+    if (CAP) {
+        rb.cap_in = p.scale / p.softcap;
+        rb.cap_out = p.softcap * 1.4426950408889634f;
+    }
 
     for (int i = 0; i < n_tiles; ++i) {
         const size_t off_now = off_ahead;                  // page of tile i + NST, looked up a pass ago
@@ -607,7 +617,7 @@ __global__ void __launch_bounds__(THREADS) attn_mma_decode_kernel(MmaAttnParams 
             __syncthreads();
         }
         zero_unfetched_rows(ring.stage_ptr(i), TILE_AT(i), src.lo_of(TILE_AT(i), key_lo), pos, warp, lane);
-        tile_step<2, true, BIAS>(qf, o, m, l, ring.stage(i), warp * 16, TILE_AT(i) * TILE, key_lo, pos, key_lo, pos, scale_log2, lane, keep, rb);
+        tile_step<2, true, BIAS, CAP>(qf, o, m, l, ring.stage(i), warp * 16, TILE_AT(i) * TILE, key_lo, pos, key_lo, pos, scale_log2, lane, keep, rb);
         __syncwarp();                                      // the warp's rows of the stage are free
         if (i + NST < n_tiles) issue_tile_rows(src, TILE_AT(i + NST), src.lo_of(TILE_AT(i + NST), key_lo), fetch_hi, ring.stage(i + NST), warp, lane, off_now);
         cp_async_commit();
@@ -797,7 +807,7 @@ __global__ void attn_mma_combine_kernel(bf16* __restrict__ out, const float* __r
 // ------------------------------------------------------------------ prefill
 // EXT: chunks, several score maps, pooled blocks, split values and float32 results (compiled out otherwise, so that the
 // plain kernel is what it was without them)
-template <bool BIAS, bool EXT>
+template <bool BIAS, bool EXT, bool CAP = false>
 __global__ void __launch_bounds__(THREADS, 3) attn_mma_prefill_kernel(MmaAttnParams p) {
     const int x_chunk = EXT ? p.chunk : 0, x_pool = EXT ? p.pool : 0, x_out_f32 = EXT ? p.out_f32 : 0;
     extern __shared__ uint8_t smem_raw[];
@@ -875,6 +885,10 @@ __global__ void __launch_bounds__(THREADS, 3) attn_mma_prefill_kernel(MmaAttnPar
         rb.r1a = rb.r1b = p.dist_r1 ? p.dist_r1[head] : 0.f;
         rb.r2a = rb.r2b = p.dist_r2 ? p.dist_r2[head] : 0.f;
     }
+    if (CAP) {
+        rb.cap_in = p.scale / p.softcap;
+        rb.cap_out = p.softcap * 1.4426950408889634f;
+    }
 
     for (int i = 0; i < n_tiles; ++i) {
         cp_async_wait<STAGES_PREFILL - 1>();
@@ -894,12 +908,12 @@ __global__ void __launch_bounds__(THREADS, 3) attn_mma_prefill_kernel(MmaAttnPar
         zero_unfetched(ring.stage_ptr(i), tile, src.lo_of(tile, key_lo), PTILE_HI(i - n_pool), tid);
         if (i - n_pool < n_kept) {
             // kept keys that lie before every row's window: all rows see the keys below `keep` and nothing else here
-            tile_step<8, true, BIAS>(qf, o, m, l, ring.stage(i), 0, p0, 0, keep - 1, 0, keep - 1, scale_log2, lane, 0, rb);
+            tile_step<8, true, BIAS, CAP>(qf, o, m, l, ring.stage(i), 0, p0, 0, keep - 1, 0, keep - 1, scale_log2, lane, 0, rb);
         } else if (p0 <= warp_hi && (p0 + TILE - 1 >= warp_lo || p0 < keep)) {   // the tile holds a key some row of the warp sees
             // every key of the tile visible to every row of the warp (most tiles of a causal prompt): no masks
             const bool all_visible = p0 + TILE - 1 <= first_pos + warp * 16 && p0 >= lo_of_row(warp_hi);
-            if (all_visible) tile_step<8, false, BIAS>(qf, o, m, l, ring.stage(i), 0, p0, lo0, hi0, lo1, hi1, scale_log2, lane, 0, rb);
-            else tile_step<8, true, BIAS>(qf, o, m, l, ring.stage(i), 0, p0, lo0, hi0, lo1, hi1, scale_log2, lane, keep, rb);
+            if (all_visible) tile_step<8, false, BIAS, CAP>(qf, o, m, l, ring.stage(i), 0, p0, lo0, hi0, lo1, hi1, scale_log2, lane, 0, rb);
+            else tile_step<8, true, BIAS, CAP>(qf, o, m, l, ring.stage(i), 0, p0, lo0, hi0, lo1, hi1, scale_log2, lane, keep, rb);
         }
         __syncthreads();
         if (i + STAGES_PREFILL < n_tiles) issue(i + STAGES_PREFILL);
@@ -955,11 +969,12 @@ LLB_API int llb_attn_mma_prefill(MmaAttnParams p, int B, int max_new, cudaStream
     dim3 grid(p.nh * (p.v_split > 1 ? p.v_split : 1), (max_new + 63) / 64, B);
     if (grid.y > 65535 || grid.z > 65535) return (int)cudaErrorInvalidValue;
     const bool ext = p.chunk > 0 || p.maps > 1 || p.v_split > 1 || p.pool > 0 || p.out_f32;
-#define LLB_PREFILL(W, BIAS, EXT)                                                                                       \
+    if (p.softcap > 0.f && (ext || p.dist_r1 || p.dist_r2 || p.q_temp_every > 0)) return (int)cudaErrorInvalidValue;
+#define LLB_PREFILL(W, ...)                                                                                             \
     do {                                                                                                                \
-        int rc = configure<W>(attn_mma_prefill_kernel<BIAS, EXT>, smem_bytes(STAGES_PREFILL));                          \
+        int rc = configure<W>(attn_mma_prefill_kernel<__VA_ARGS__>, smem_bytes(STAGES_PREFILL));                         \
         if (rc) return rc;                                                                                              \
-        llb_launch(attn_mma_prefill_kernel<BIAS, EXT>, grid, dim3(THREADS), smem_bytes(STAGES_PREFILL), stream, p);     \
+        llb_launch(attn_mma_prefill_kernel<__VA_ARGS__>, grid, dim3(THREADS), smem_bytes(STAGES_PREFILL), stream, p);     \
         return llb_status();                                                                                            \
     } while (0)
     if (p.dist_r1 || p.dist_r2 || p.q_temp_every > 0) {          // scores that depend on the positions themselves
@@ -967,6 +982,7 @@ LLB_API int llb_attn_mma_prefill(MmaAttnParams p, int B, int max_new, cudaStream
         if (ext) LLB_PREFILL(4, true, true);
         LLB_PREFILL(2, true, false);
     }
+    if (p.softcap > 0.f) LLB_PREFILL(6, false, false, true);
     if (ext) LLB_PREFILL(5, false, true);
     LLB_PREFILL(0, false, false);
 #undef LLB_PREFILL
@@ -1004,14 +1020,14 @@ LLB_API int llb_attn_mma_decode_max_clusters(int size) {
 LLB_DEFINE_SET_STAMPS
 
 namespace {
-template <bool BIAS>
+template <bool BIAS, bool CAP = false>
 int launch_decode(MmaAttnParams p, int B, cudaStream_t stream) {
     int G = p.nh / p.nkvh;
     dim3 grid(p.n_splits, p.nkvh * ((G + 15) / 16), B);
     if (grid.y > 65535 || grid.z > 65535) return (int)cudaErrorInvalidValue;
-    auto kernel = attn_mma_decode_kernel<STAGES, BIAS>;
+    auto kernel = attn_mma_decode_kernel<STAGES, BIAS, CAP>;
     const int smem = smem_bytes_decode(STAGES);
-    int rc = configure<BIAS ? 3 : 1>(kernel, smem);
+    int rc = configure<CAP ? 7 : BIAS ? 3 : 1>(kernel, smem);
     if (rc) return rc;
     if (p.cluster && p.n_splits > 8) {
         static bool allowed = false;
@@ -1061,7 +1077,9 @@ LLB_API int llb_attn_mma_decode(MmaAttnParams p, int B, cudaStream_t stream) {
     if (p.cluster && p.n_splits > MAX_CLUSTER) return (int)cudaErrorInvalidValue;
     if (p.dist_r1 || p.dist_r2 || p.q_temp_every > 0) {          // scores that depend on the positions themselves
         if (!p.dist_r1 != !p.dist_r2) return (int)cudaErrorInvalidValue;
+        if (p.softcap > 0.f) return (int)cudaErrorInvalidValue;
         return launch_decode<true>(p, B, stream);
     }
+    if (p.softcap > 0.f) return launch_decode<false, true>(p, B, stream);
     return launch_decode<false>(p, B, stream);
 }

@@ -18,7 +18,8 @@
 // head (several score maps over one set of values) and a cache key row holds their keys side by side.  `pool` P > 0 (with a
 // window W): beside the window's keys, one key and value per block of P positions that lies wholly before the window
 // (block b is seen from p when b P + P - 1 <= p - W), read at row b of a second cache and walked before the window's tiles;
-// tokens and blocks share one softmax.  `out_f32`: the result is float32 whatever the operands are.
+// tokens and blocks share one softmax.  `out_f32`: the result is float32 whatever the operands are.  `softcap` c > 0: a
+// (scaled) score s becomes c tanh(s / c); a sink is not capped.
 //
 // Keys are walked in tiles of one cache page with an online softmax, so nothing of size
 // [queries, keys] is ever stored.
@@ -89,6 +90,7 @@ struct AttnParams {
     const void* pool_v;   // [pages, nkvh / maps, LLB_PAGE, DV]
     const int* pool_table;  // [B, pool_table_stride]
     int pool_table_stride;
+    float softcap;        // > 0: scaled scores pass through softcap * tanh(. / softcap)
 };
 
 template <typename T, bool DECODE>
@@ -305,8 +307,14 @@ __global__ void __launch_bounds__(WARPS * 32) attn_kernel(AttnParams p) {
                 v0 = kp0 < blocks_seen;
                 v1 = kp1 < blocks_seen;
             }
-            s0 = v0 ? s0 * row_scale : -INFINITY;
-            s1 = v1 ? s1 * row_scale : -INFINITY;
+            s0 *= row_scale;
+            s1 *= row_scale;
+            if (p.softcap > 0.f) {
+                s0 = p.softcap * tanhf(s0 / p.softcap);
+                s1 = p.softcap * tanhf(s1 / p.softcap);
+            }
+            s0 = v0 ? s0 : -INFINITY;
+            s1 = v1 ? s1 : -INFINITY;
             if (p.dist_r1 && !pooled) {
                 if (v0) s0 -= r1 * log1pf(r2 * (float)(pos - kp0));
                 if (v1) s1 -= r1 * log1pf(r2 * (float)(pos - kp1));

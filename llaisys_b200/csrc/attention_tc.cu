@@ -1,7 +1,8 @@
 // bfloat16 prefill attention over the paged cache on the 5th-generation tensor cores (tcgen05),
 // for head sizes 64 and 128.  Same formula and masks as attention_simt.cu (xsmccc/llaisys
 // src/ops/self_attention/cpu/self_attention_cpu.cpp:28-112, plus the window, the first keys that stay visible
-// behind a window, and the value-less sink term e^0 in the softmax's denominator).  All keys, those of
+// behind a window, the value-less sink term in the softmax's denominator, of score 0 or learned per head, and a cap on the
+// scores, c tanh(s / c)).  All keys, those of
 // the step included, are read from the cache: the caller appends before it attends.
 //
 // A CTA owns 128 consecutive new tokens of one query head.  Warps 0-3 are the softmax warps:
@@ -77,6 +78,8 @@ struct TcAttnParams {
     int n_split;                // 1, 2 or 4: CTAs (a thread-block cluster) that share the key range of a row block
     int keep_first;             // with a window: keys before this position stay visible
     int sink;                   // the softmax's denominator has one more term e^0 (no value)
+    const float* sink_logits;   // [nh] or null: that term is e^(sink_logits[head]) instead (implies a sink)
+    float softcap;              // > 0: scaled scores pass through softcap * tanh(. / softcap)
 };
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -197,6 +200,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
+template <bool CAP>
 __global__ void __launch_bounds__(THREADS, 2)
 attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, TcAttnParams p) {
@@ -273,8 +277,8 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     llb_grid_dependency_sync();
     bool failed = false;
     float m = -INFINITY, l = 0.f;                                   // row threads: the exponent base of the row, its sum
-    if (p.sink && rank == 0) {                                      // the sink's term e^0, once per row
-        m = 0.f;
+    if ((p.sink || p.sink_logits) && rank == 0) {                   // the sink's term, once per row (m is on the base-2 scale)
+        m = p.sink_logits ? p.sink_logits[head] * 1.4426950408889634f : 0.f;
         l = 1.f;
     }
     const uint32_t lane_addr = tmem + ((uint32_t)((warp & 3) * 32) << 16);
@@ -387,8 +391,9 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         // ================================================= softmax: thread r owns query row r
         const int qpos = first_pos + min(tid, n_rows - 1);          // rows past the end behave like the last row
         const int qlo = p.window > 0 ? max(0, qpos - p.window + 1) : 0;
-        const float scale_log2 = p.scale * 1.4426950408889634f;
+        const float scale_log2 = CAP ? 1.f : p.scale * 1.4426950408889634f;       // capped scores arrive on the base-2 scale
         const uint64_t scale2 = twice(scale_log2);
+        const float cap_in = CAP ? p.scale / p.softcap : 0.f, cap_out = CAP ? p.softcap * 1.4426950408889634f : 0.f;
 
         for (int i = 0; i < n_tiles && !failed; ++i) {
             const int s = i % KV_STAGES;
@@ -400,6 +405,10 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             for (int c = 0; c < BKV; c += 16) tmem_ld16_nowait(lane_addr + s * BKV + c, sr + c);
             tmem_wait();
 
+            if (CAP) {
+#pragma unroll
+                for (int j = 0; j < BKV; ++j) sr[j] = __float_as_uint(cap_out * llb_tanh_fast(__uint_as_float(sr[j]) * cap_in));
+            }
             // ---- mask (only tiles that some row of the block sees in part), maximum
             if (it_lo + i < n_kept) {                                // a tile of kept keys before every row's window
 #pragma unroll
@@ -626,17 +635,18 @@ LLB_API int llb_attn_tc_prefill(const void* q, int T, int row_stride, const void
     if (rc) return rc;
     rc = llb_tma::bf16_map_64(vpool, (long long)n_pages * p.nkvh * BKV, DH, DH, BKV, &mv);
     if (rc) return rc;
-    static bool configured = false;
-    if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_tc_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
+    auto kernel = p.softcap > 0.f ? attn_tc_prefill_kernel<true> : attn_tc_prefill_kernel<false>;
+    static bool configured[2] = {false, false};
+    if (!configured[p.softcap > 0.f]) {
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES);
         if (e != cudaSuccess) return -2000 - (int)e;
-        configured = true;
+        configured[p.softcap > 0.f] = true;
     }
     if (p.n_split == 1) {
-        llb_launch(attn_tc_prefill_kernel, grid, dim3(THREADS), SMEM_BYTES, stream, mq, mk, mv, p);
+        llb_launch(kernel, grid, dim3(THREADS), SMEM_BYTES, stream, mq, mk, mv, p);
         return llb_status();
     }
-    llb_prefer_max_shared((const void*)attn_tc_prefill_kernel);
+    llb_prefer_max_shared((const void*)kernel);
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = dim3(THREADS);
@@ -656,6 +666,6 @@ LLB_API int llb_attn_tc_prefill(const void* q, int T, int row_stride, const void
     ++n_attr;
     cfg.attrs = attr;
     cfg.numAttrs = n_attr;
-    cudaLaunchKernelEx(&cfg, attn_tc_prefill_kernel, mq, mk, mv, p);
+    cudaLaunchKernelEx(&cfg, kernel, mq, mk, mv, p);
     return llb_status();
 }

@@ -94,6 +94,14 @@ __device__ __forceinline__ bool paged_survives(int lp, int last_lp, int ring, in
     return lp < pinned || lp + ring > last_lp;
 }
 
+// tanh(x) = 1 - 2 / (1 + e^(2 x)) by the special-function unit; absolute error a few 2^-23.  For score caps of bfloat16 kernels.
+__device__ __forceinline__ float llb_tanh_fast(float x) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.0f));
+    return fmaf(-2.0f, r, 1.0f);
+}
+
 static inline int llb_status() { return (int)cudaGetLastError(); }
 
 // ---- programmatic dependent launch

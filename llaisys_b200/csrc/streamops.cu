@@ -5,8 +5,10 @@
 //   branch_mean   out[r] = mult * sum_b x_b[r] / sqrt(mean(x_b[r]^2) + eps) * w_b: several mixers' results, each normed
 //                 over the row with a weight of its own, averaged
 //   scale_rows    x *= c
+//   layer_norm    out[r] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * weight, v = x[rows ? rows[r] : r]
+//   copy_rows     rows of the stream, converted, into a matrix of another row stride
 //
-// One block per row; a row is read once (it is kept in shared memory between the sum of squares and the output).
+// One block (layer_norm of many rows: one warp) per row; a row is read once.
 #include "common.cuh"
 
 __device__ __forceinline__ float block_sum_256(float v, float* red) {
@@ -154,6 +156,146 @@ LLB_API int llb_branch_mean(BranchMeanParams p, int w_dtype, int T, cudaStream_t
     if (T == 0) return 0;
     if (p.n < 1 || p.n > 4) return (int)cudaErrorInvalidValue;
     LLB_DISPATCH_DTYPE(w_dtype, TW, llb_launch(branch_mean_kernel<TW>, dim3(T), dim3(256), 0, stream, p));
+    return llb_status();
+}
+
+// ------------------------------------------------------------------ layer norm
+// The mean first, then the squares of the deviations from it, both over the row in registers (or, for widths that are no
+// multiple of 4 or beyond 16,384, in shared memory).  TPR threads share a row; a thread holds PER pieces of 16 bytes.
+template <int TPR>
+__device__ __forceinline__ float row_sum(float v, float* red) {
+    v = warp_sum(v);
+    if (TPR == 32) return v;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    __syncthreads();
+    if (lane == 0) red[warp] = v;
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) s += red[w];
+    return s;
+}
+
+template <typename TW, typename TO, int TPR, int PER>
+__global__ void __launch_bounds__(256) layer_norm_kernel(const float* __restrict__ x, const TW* __restrict__ weight, TO* __restrict__ out,
+                                                         const int* __restrict__ rows, int R, int H, float eps) {
+    __shared__ float red[8];
+    const int tid = threadIdx.x % TPR, r = blockIdx.x * (256 / TPR) + threadIdx.x / TPR;
+    llb_grid_dependency_sync();
+    if (r >= R) return;                                    // (whole warps or whole blocks)
+    const float* src = x + (size_t)(rows ? rows[r] : r) * H;
+    float4 v[PER];
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int j = (tid + i * TPR) * 4;
+        v[i] = j < H ? *reinterpret_cast<const float4*>(src + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    }
+    const float mean = row_sum<TPR>(s, red) / (float)H;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        if ((tid + i * TPR) * 4 >= H) continue;
+        v[i].x -= mean;
+        v[i].y -= mean;
+        v[i].z -= mean;
+        v[i].w -= mean;
+        ss += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+    }
+    const float inv = 1.0f / sqrtf(row_sum<TPR>(ss, red) / (float)H + eps);
+    TO* dst = out + (size_t)r * H;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int j = (tid + i * TPR) * 4;
+        if (j >= H) continue;
+        const float y[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
+        alignas(16) TO o[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[e] = from_f32<TO>(y[e] * inv * to_f32(weight[j + e]));
+        if constexpr (sizeof(TO) == 4) *reinterpret_cast<float4*>(dst + j) = *reinterpret_cast<const float4*>(o);
+        else *reinterpret_cast<uint2*>(dst + j) = *reinterpret_cast<const uint2*>(o);
+    }
+}
+
+template <typename TW, typename TO>
+__global__ void __launch_bounds__(256) layer_norm_any_kernel(const float* __restrict__ x, const TW* __restrict__ weight, TO* __restrict__ out,
+                                                             const int* __restrict__ rows, int H, float eps) {
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[8];
+    const int r = blockIdx.x;
+    llb_grid_dependency_sync();
+    const float* src = x + (size_t)(rows ? rows[r] : r) * H;
+    float s = 0.f;
+    for (int i = threadIdx.x; i < H; i += 256) s += row[i] = src[i];
+    const float mean = block_sum_256(s, red) / (float)H;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < H; i += 256) ss = fmaf(row[i] - mean, row[i] - mean, ss);
+    const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += 256) out[(size_t)r * H + i] = from_f32<TO>((row[i] - mean) * inv * to_f32(weight[i]));
+}
+
+template <typename TW, typename TO>
+static int layer_norm_launch(const float* x, const TW* w, TO* out, const int* rows, int R, int H, float eps, cudaStream_t stream) {
+    if (H % 4 == 0 && H <= 16384 && !(((uintptr_t)x | (uintptr_t)out) & 15)) {
+#define LLB_LN(TPR, PER) do { llb_launch(layer_norm_kernel<TW, TO, TPR, PER>, dim3((R + 256 / TPR - 1) / (256 / TPR)), dim3(256), 0,     \
+                                         stream, x, w, out, rows, R, H, eps); return llb_status(); } while (0)
+        if (R >= 256) {                                    // many rows: a warp per row
+            if (H <= 512) LLB_LN(32, 4);
+            if (H <= 1024) LLB_LN(32, 8);
+            if (H <= 2048) LLB_LN(32, 16);
+            if (H <= 4096) LLB_LN(32, 32);
+        }
+        if (H <= 1024) LLB_LN(256, 1);
+        if (H <= 2048) LLB_LN(256, 2);
+        if (H <= 4096) LLB_LN(256, 4);
+        LLB_LN(256, 16);
+#undef LLB_LN
+    }
+    const size_t smem = (size_t)H * sizeof(float);
+    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+    auto k = layer_norm_any_kernel<TW, TO>;
+    static bool configured = false;
+    if (!configured && smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        if (e != cudaSuccess) return (int)e;
+        configured = true;
+    }
+    llb_launch(k, dim3(R), dim3(256), smem, stream, x, w, out, rows, H, eps);
+    return llb_status();
+}
+
+LLB_API int llb_layer_norm(const float* x, const void* weight, int w_dtype, void* out, int out_dtype, const int* rows, int R, int H,
+                           float eps, cudaStream_t stream) {
+    if (R == 0) return 0;
+    LLB_DISPATCH_DTYPE(w_dtype, TW, {
+        LLB_DISPATCH_DTYPE(out_dtype, TO, { return layer_norm_launch<TW, TO>(x, (const TW*)weight, (TO*)out, rows, R, H, eps, stream); });
+    });
+    return 0;
+}
+
+// ------------------------------------------------------------------ rows of the stream into another matrix
+template <typename TO>
+__global__ void __launch_bounds__(256) copy_rows_kernel(const float* __restrict__ x, TO* __restrict__ out, int ld, int H) {
+    llb_grid_dependency_sync();
+    const float* src = x + (size_t)blockIdx.x * H;
+    TO* dst = out + (size_t)blockIdx.x * ld;
+    const bool vec = H % 4 == 0 && ld % 4 == 0 && !(((uintptr_t)x | (uintptr_t)out) & 15);
+    if (vec) {
+        for (int i = threadIdx.x * 4; i < H; i += 1024) {
+            const float4 v = *reinterpret_cast<const float4*>(src + i);
+            alignas(16) TO o[4] = {from_f32<TO>(v.x), from_f32<TO>(v.y), from_f32<TO>(v.z), from_f32<TO>(v.w)};
+            if constexpr (sizeof(TO) == 4) *reinterpret_cast<float4*>(dst + i) = *reinterpret_cast<const float4*>(o);
+            else *reinterpret_cast<uint2*>(dst + i) = *reinterpret_cast<const uint2*>(o);
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < H; i += 256) dst[i] = from_f32<TO>(src[i]);
+}
+
+LLB_API int llb_copy_rows(const float* x, void* out, int out_dtype, int ld, int T, int H, cudaStream_t stream) {
+    if (T == 0) return 0;
+    LLB_DISPATCH_DTYPE(out_dtype, TO, llb_launch(copy_rows_kernel<TO>, dim3(T), dim3(256), 0, stream, x, (TO*)out, ld, H));
     return llb_status();
 }
 

@@ -1,5 +1,6 @@
 """Python faces of csrc/headops.cu (norm, rotation and cache append of packed heads; pooled blocks; the difference of two
-score maps) and csrc/streamops.cu (gated joins of the residual stream, the mean of normed branches, a scale)."""
+score maps) and csrc/streamops.cu (gated joins of the residual stream, the mean of normed branches, layer norm, copies of
+rows, a scale)."""
 from __future__ import annotations
 
 import ctypes
@@ -158,3 +159,25 @@ def scale_(x: torch.Tensor, c: float) -> torch.Tensor:
     f = _fn(load_module("streamops.cu"), "llb_scale_rows", [c_void_p, c_longlong, c_float, c_void_p])
     _check(f(_ptr(x), x.numel(), c, _stream()), "scale")
     return x
+
+
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """(x - mean) / sqrt(mean((x - mean)^2) + eps) * weight over the rows of the float32 stream x [T, H], in out_dtype; with
+    rows (int32) only those rows, [len(rows), H]."""
+    _need_cuda(x, weight, rows)
+    T, H = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and weight.numel() == H and weight.is_contiguous()
+    R = T if rows is None else rows.numel()
+    out = torch.empty((R, H), dtype=out_dtype, device=x.device)
+    f = _fn(load_module("streamops.cu"), "llb_layer_norm", [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_float,
+                                                            c_void_p])
+    _check(f(_ptr(x), _ptr(weight), _dt(weight), _ptr(out), DT[out_dtype], _ptr(rows), R, H, eps, _stream()), "layer norm")
+    return out
+
+
+def copy_rows(x: torch.Tensor, out: torch.Tensor) -> None:
+    """The rows of the float32 stream x [T, H], converted, into out [T, H] (a view with any row stride)."""
+    _need_cuda(x, out)
+    assert x.dtype == torch.float32 and x.is_contiguous() and out.shape == x.shape and out.stride(1) == 1
+    f = _fn(load_module("streamops.cu"), "llb_copy_rows", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(x), _ptr(out), _dt(out), out.stride(0), x.shape[0], x.shape[1], _stream()), "copy of rows")

@@ -698,7 +698,7 @@ class _AttnParams(ctypes.Structure):
                 ("sink_logits", c_void_p), ("v_in_k", c_int), ("kv_row_stride", c_int),
                 ("dist_r1", c_void_p), ("dist_r2", c_void_p), ("q_temp_coef", c_float), ("q_temp_every", c_int),
                 ("chunk", c_int), ("maps", c_int), ("out_f32", c_int), ("pool", c_int), ("pool_k", c_void_p), ("pool_v", c_void_p),
-                ("pool_table", c_void_p), ("pool_table_stride", c_int)]
+                ("pool_table", c_void_p), ("pool_table_stride", c_int), ("softcap", c_float)]
 
 
 class _MmaAttnParams(ctypes.Structure):
@@ -712,7 +712,7 @@ class _MmaAttnParams(ctypes.Structure):
                 ("keep_first", c_int), ("pinned", c_int), ("sink", c_int), ("sink_logits", c_void_p),
                 ("dist_r1", c_void_p), ("dist_r2", c_void_p), ("q_temp_coef", c_float), ("q_temp_every", c_int),
                 ("chunk", c_int), ("maps", c_int), ("out_f32", c_int), ("v_split", c_int), ("pool", c_int), ("pool_k", c_void_p),
-                ("pool_v", c_void_p), ("pool_table", c_void_p), ("pool_table_stride", c_int)]
+                ("pool_v", c_void_p), ("pool_table", c_void_p), ("pool_table_stride", c_int), ("softcap", c_float)]
 
 
 MMA_ATTENTION = True                         # tests switch the tensor-core attention off to compare
@@ -751,7 +751,7 @@ def decode_fusion_ok(dtype: torch.dtype, dh: int) -> bool:
 class _TcAttnParams(ctypes.Structure):
     _fields_ = [("out", c_void_p), ("page_table", c_void_p), ("table_stride", c_int), ("seq_start", c_void_p),
                 ("seq_len_before", c_void_p), ("nh", c_int), ("nkvh", c_int), ("window", c_int), ("scale", c_float),
-                ("err", c_void_p), ("n_split", c_int), ("keep_first", c_int), ("sink", c_int)]
+                ("err", c_void_p), ("n_split", c_int), ("keep_first", c_int), ("sink", c_int), ("sink_logits", c_void_p), ("softcap", c_float)]
 
 
 TC_ATTENTION = True                          # tests switch the tcgen05 prefill attention off to compare
@@ -802,7 +802,10 @@ class AttnExtras:
     and value head (h / (nh / nkvh)) / maps, and a cache key row holds the maps' keys side by side); `out_f32` (the result
     is float32 whatever the operands are); `pool` = (P, blocks): beside the keys of a window W, one key and value per block
     of P positions that lies wholly before the window (block b is seen from position p when b P + P - 1 <= p - W), read
-    at row b of the cache view `blocks`; tokens and blocks share one softmax."""
+    at row b of the cache view `blocks`; tokens and blocks share one softmax.
+
+    `softcap` c (> 0): a scaled score s becomes c tanh(s / c) (a sink is not capped); on every attention kernel, but not together
+    with a distance penalty, a query temperature or the four options above on the tensor cores."""
     value_dim: Optional[int] = None
     keep_first: int = 0
     pinned: int = 0
@@ -814,10 +817,11 @@ class AttnExtras:
     maps: int = 1
     out_f32: bool = False
     pool: Optional[tuple] = None
+    softcap: float = 0.0
 
     def plain(self, dh: int) -> bool:
         return (self.value_dim in (None, dh) and not self.keep_first and not self.pinned and not self.sink
-                and self.sink_logits is None and not self.positional() and not self.cuda_core_only())
+                and self.sink_logits is None and not self.softcap and not self.positional() and not self.cuda_core_only())
 
     def cuda_core_only(self) -> bool:
         """True with an option that only the CUDA-core kernel (and the mma.sync prefill kernel) has."""
@@ -837,6 +841,7 @@ def _attn_params(qkv, out, nh, nkvh, dh, kpool, vpool, page_table, ring, seq_sta
     p.v_new = qkv.data_ptr() + (nh + nkvh) * dh * es
     if extras is not None:
         p.keep_first, p.pinned, p.sink = (extras.keep_first if window else 0), extras.pinned, int(extras.sink)
+        p.softcap = float(extras.softcap)
         if extras.sink_logits is not None:
             assert extras.sink_logits.dtype == torch.float32 and extras.sink_logits.numel() == nh
             p.sink_logits = extras.sink_logits.data_ptr()
@@ -905,13 +910,16 @@ def attention_prefill(qkv, nh, nkvh, dh, kpool, vpool, page_table, ring, seq_sta
 
 
 def _attention_prefill_tc(qkv, out, nh, nkvh, dh, kpool, vpool, page_table, seq_start, seq_len_before, n_seqs, max_new,
-                          window, scale, tc_split=0, keep_first=0, sink=False):
+                          window, scale, tc_split=0, keep_first=0, sink=False, sink_logits=None, softcap=0.0):
     """The tcgen05 prefill kernel (csrc/attention_tc.cu): every key from a cache that keeps them all."""
     p = _TcAttnParams()
     p.out, p.page_table, p.table_stride = out.data_ptr(), page_table.data_ptr(), page_table.shape[1]
     p.seq_start, p.seq_len_before = seq_start.data_ptr(), seq_len_before.data_ptr()
     p.nh, p.nkvh, p.window, p.scale = nh, nkvh, int(window or 0), scale
     p.keep_first, p.sink = (int(keep_first) if window else 0), int(sink)
+    p.sink_logits, p.softcap = _ptr(sink_logits), float(softcap)
+    if sink_logits is not None:
+        assert sink_logits.dtype == torch.float32 and sink_logits.numel() == nh
     p.err = _tc_resources(qkv.device)[2].data_ptr()
     # few row blocks (up to one and a half per SM): two CTAs share each block's key range, so that the longest
     # CTA gets shorter (measured at 12 heads: 30.5 vs 33.7 us at 2,048 tokens, 73 vs 64 us at 4,096; four CTAs
@@ -978,13 +986,13 @@ def _attention_extras(decode, qkv, nh, nkvh, dh, kpool, vpool, page_table, ring,
     out = torch.empty((qkv.shape[0], nh * dv), dtype=torch.float32 if extras.out_f32 else qkv.dtype, device=qkv.device)
     only_simt = extras.cuda_core_only()
     if (not only_simt and not decode and dv == dh and all_from_cache and prefill_tc_ok(qkv.dtype, dh) and not extras.pinned and scale > 0
-            and extras.sink_logits is None and not extras.positional()
+            and not extras.positional()
             and ring >= page_table.shape[1] and qkv.stride(0) % 8 == 0):
         # a cache that keeps every key, head size 64 or 128: the tcgen05 prefill kernel, as for the plain attention
         _attention_prefill_tc(qkv, out, nh, nkvh, dh, kpool, vpool, page_table, seq_start, seq_len_before, n_seqs, max_new,
-                              window, scale, 0, extras.keep_first, extras.sink)
+                              window, scale, 0, extras.keep_first, extras.sink, extras.sink_logits, extras.softcap)
         return out
-    if (only_simt and not decode and prefill_ext_ok(qkv, dh, dv) and not extras.keep_first and not extras.sink
+    if (only_simt and not extras.softcap and not decode and prefill_ext_ok(qkv, dh, dv) and not extras.keep_first and not extras.sink
             and extras.sink_logits is None and (extras.pool is None or not extras.positional())
             and not ((kpool.data_ptr() | vpool.data_ptr() | out.data_ptr()) & 15)):
         # prompts in bfloat16: the mma.sync prefill kernel with its extensions (a block owns one half of values twice as
@@ -995,7 +1003,7 @@ def _attention_extras(decode, qkv, nh, nkvh, dh, kpool, vpool, page_table, ring,
         f = _fn(_mma_lib(dh), "llb_attn_mma_prefill", [_MmaAttnParams, c_int, c_int, c_void_p])
         _check(f(p, n_seqs, max_new, _stream()), "attention_prefill (tensor cores)")
         return out
-    if not only_simt and dv == dh and _mma_ok(qkv, dh):
+    if not only_simt and dv == dh and _mma_ok(qkv, dh) and not (extras.softcap and extras.positional()):
         # keys and values of one width that the tensor-core kernel takes: the same kernels as the plain attention
         # (a distance penalty and a query temperature are applied to the score fragments in registers)
         p = _attn_params(qkv, out, nh, nkvh, dh, kpool, vpool, page_table, ring, seq_start, seq_len_before, window, scale,

@@ -56,14 +56,38 @@ class ParallelResidual(Block):
         hs = []
         for i in range(0, len(norms), 2):
             hs += kernels.rmsnorm_multi(residual, [n.weight for n in norms[i:i + 2]], norms[0].eps, self.env.dtype)
-        mixers = iter(users)
-        for sub, h in zip(self.sublayers, hs):
-            if sub.category == "mixer":
-                call = next(mixers)
-                if not sub.part.forward_into(h, ctx, call, residual):
-                    kernels.residual_add(residual, sub.part.forward(h, ctx, call))
-            elif not sub.part.forward_into(h, ctx, residual):
-                kernels.residual_add(residual, sub.part.forward(h, ctx))
+        _add_branches(self.sublayers, hs, residual, ctx, users)
+        return residual, None
+
+
+def _add_branches(sublayers, hs, residual, ctx, users):
+    """residual += sum over the sub-layers of part(h): each adds in its own last kernel where it can."""
+    from .. import kernels
+    mixers = iter(users)
+    for sub, h in zip(sublayers, hs):
+        if sub.category == "mixer":
+            call = next(mixers)
+            if not sub.part.forward_into(h, ctx, call, residual):
+                kernels.residual_add(residual, sub.part.forward(h, ctx, call))
+        elif not sub.part.forward_into(h, ctx, residual):
+            kernels.residual_add(residual, sub.part.forward(h, ctx))
+
+
+@register_part("block", "shared_norm_parallel")
+class SharedNormParallel(Block):
+    """x -> x + sum over the sub-layers of part(h), h = norm(x): one norm, the first sub-layer's, serves all of them (of any
+    kind).  Once the norm has run the parts may add into the stream in any order, each in its own last kernel where it
+    can."""
+    capturable = True
+
+    def __init__(self, sublayers, env, params=None):
+        super().__init__(sublayers, env, params)
+        if self.sublayers[0].norm is None or any(sub.norm is not None for sub in self.sublayers[1:]):
+            raise ValueError("the layer's one norm stands before its first sub-layer")
+
+    def forward(self, residual, pending, ctx, users):
+        h = settle(residual, pending, self.sublayers[0].norm)
+        _add_branches(self.sublayers, [h] * len(self.sublayers), residual, ctx, users)
         return residual, None
 
 

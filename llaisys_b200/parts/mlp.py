@@ -51,11 +51,12 @@ class SwiGLUMLP(FeedForward):
 
 @register_part("ffn", "gated_mlp")
 class GatedMLP(FeedForward):
-    """down(act(gate(x)) * up(x)) with the activation a parameter: "silu", "relu" or "gelu_tanh".  The gate
+    """down(act(gate(x)) * up(x)) with the activation a parameter: "silu", "relu", "gelu_tanh", or "swish_clamped":
+    g = min(gate(x), limit), u = clamp(up(x), -limit, limit), down(g sigmoid(alpha g) (u + 1)).  The gate
     and up matrices are kept as one [2I, H] matrix so that one product serves both; the activation and the product of
     the halves are one pass in float32.  With `bias` every projection has a bias (tensors named after the matrices with
     `bias_suffix`, default ".b").  The result is returned in float32 (it may be normed or scaled before it joins the
-    stream).  params: hidden_size, intermediate_size, act, bias, bias_suffix, names (local tensor names of gate, up, down)."""
+    stream) unless the part is asked to add it to the stream itself.  params: hidden_size, intermediate_size, act, limit and alpha (swish_clamped), bias, bias_suffix, names (local tensor names of gate, up, down)."""
     capturable = True
 
     def __init__(self, spec, env):
@@ -64,6 +65,9 @@ class GatedMLP(FeedForward):
         self.hidden, self.inter, self.act = int(p["hidden_size"]), int(p["intermediate_size"]), str(p.get("act", "silu"))
         if self.act not in kernels.ops.GLU_ACTS:
             raise ValueError(f"unknown activation {self.act!r}; known: {sorted(kernels.ops.GLU_ACTS)}")
+        self.limit, self.alpha = float(p.get("limit", float("inf"))), float(p.get("alpha", 1.0))
+        if not self.limit > 0:
+            raise ValueError(f"the limit must be positive, got {self.limit}")
         self.names = dict({"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}, **(p.get("names") or {}))
         self.bias, self.bias_suffix = bool(p.get("bias", False)), str(p.get("bias_suffix", ".b"))
         self.gate_up = self.down = self.b_gate_up = self.b_down = None
@@ -88,12 +92,20 @@ class GatedMLP(FeedForward):
             self.b_gate_up = torch.cat([tensors[self.names["gate"] + b].float(), tensors[self.names["up"] + b].float()]).contiguous()
             self.b_down = tensors[self.names["down"] + b].float().contiguous()
 
-    def forward(self, x, ctx):
+    def _activated(self, x):
         if self.act == "silu" and not self.bias:
-            act = kernels.linear_swiglu(x, self.gate_up)
-        else:
-            act = kernels.glu(kernels.linear(x, self.gate_up, self.b_gate_up), self.act)
+            return kernels.linear_swiglu(x, self.gate_up)
+        return kernels.glu(kernels.linear(x, self.gate_up, self.b_gate_up), self.act, limit=self.limit, alpha=self.alpha)
+
+    def forward(self, x, ctx):
+        act = self._activated(x)
         return kernels.linear(act, self.down, self.b_down, out_dtype=delta_dtype(act))
+
+    def forward_into(self, x, ctx, residual):
+        if not kernels.linear_into_ok(x.new_empty((x.shape[0], self.inter)), self.down, self.b_down, residual):
+            return False
+        kernels.linear_into(self._activated(x), self.down, self.b_down, residual)
+        return True
 
 
 def delta_dtype(x):

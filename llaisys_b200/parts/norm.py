@@ -47,3 +47,27 @@ class RMSNorm(Norm):
             raise ValueError("the norm that follows must be an RMS norm with the same eps")
         return kernels.scaled_norm_add(residual, delta, self.weight, float(mult), then.weight if then is not None else None,
                                        self.eps, 0.0, self.env.dtype)
+
+
+@register_part("norm", "layer_norm")
+class LayerNorm(Norm):
+    """y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w over a row, without a bias.  params: size, eps, tensor (the
+    weight's local name, "weight" unless given; "" when the tensor carries the part's own name)."""
+    capturable = True
+
+    def __init__(self, spec, env):
+        super().__init__(spec, env)
+        self.size, self.eps = int(spec.params["size"]), float(spec.params["eps"])
+        self.tensor = str(spec.params.get("tensor", "weight"))
+        self.weight = None
+
+    def tensors(self):
+        return {self.tensor: TensorDecl((self.size,), init="one_plus_normal", use="vector")}
+
+    def load(self, tensors):
+        self.weight = tensors[self.tensor].contiguous()
+
+    def forward(self, residual, delta=None, rows=None):
+        if delta is not None:
+            kernels.residual_add(residual, delta)
+        return kernels.layer_norm(residual, self.weight, self.eps, self.env.dtype, rows=rows)

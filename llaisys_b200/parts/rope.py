@@ -66,13 +66,28 @@ class RotaryHalfSplit(PositionEncoding):
                             tok_pos=ctx.tok_pos, err=ctx.err)
 
 
-def _leading_tables(dims: int, base: float, device, rows: int, factor: float = 1.0):
-    key = ("leading", dims, base, str(device)) + ((factor,) if factor != 1.0 else ())
+def wavelength_frequencies(dims: int, base: float, wave):
+    """float64 frequencies [dims / 2] of a rotation, base^(-2i/dims), rescaled by their wavelengths 2 pi / f with
+    wave = {factor, low, high, original} (None: as they are): a wavelength below original / high keeps its frequency, one
+    above original / low has it divided by factor, and between the two f becomes (1 - s) f / factor + s f with
+    s = (original / wavelength - low) / (high - low)."""
+    import math
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / dims)
+    if not wave:
+        return f
+    factor, low, high, original = (float(wave[k]) for k in ("factor", "low", "high", "original"))
+    length = 2.0 * math.pi / f
+    s = (original / length - low) / (high - low) if high != low else torch.ones_like(f)
+    out = torch.where(length < original / high, f, (1.0 - s) * f / factor + s * f)
+    return torch.where(length > original / low, f / factor, out)
+
+
+def _leading_tables(dims: int, base: float, device, rows: int, factor: float = 1.0, wave=None):
+    key = ("leading", dims, base, str(device)) + ((factor,) if factor != 1.0 else ()) + (tuple(sorted(wave.items())) if wave else ())
     have = _TABLES.get(key)
     if have is None or have[0].shape[0] < rows:
-        half = dims // 2
-        i = torch.arange(half, dtype=torch.float64)
-        freq = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / dims) / factor
+        freq = wavelength_frequencies(dims, base, wave) / factor
         ang = torch.arange(rows, dtype=torch.float64)[:, None] * freq[None, :]
         have = (torch.cos(ang).to(torch.float32).to(device).contiguous(), torch.sin(ang).to(torch.float32).to(device).contiguous())
         _TABLES[key] = have
@@ -87,7 +102,7 @@ class RotaryLeading(PositionEncoding):
     encodes nothing.  Tables [positions, dims/2] are built in float64 on the host and kept in float32, sized once by
     prepare().  Mixers that rotate in their own kernels take the tables through pair_tables(); `pair_layout` tells them
     which dimensions pair up.  params: head_dim, dims, base, factor (default 1: every frequency is divided by it, the
-    linear stretching of positions)."""
+    linear stretching of positions), wave (None, or what wavelength_frequencies() rescales by)."""
     capturable = True
     pair_layout = "halves"
 
@@ -99,6 +114,7 @@ class RotaryLeading(PositionEncoding):
             raise ValueError(f"the frequencies' divisor must be positive, got {self.factor}")
         if self.dims % 2 or not (0 <= self.dims <= self.head_dim):
             raise ValueError(f"rotated dimensions must be even and at most the head size {self.head_dim}, got {self.dims}")
+        self.wave = {k: float(v) for k, v in spec.params["wave"].items()} if spec.params.get("wave") else None
         self._tables = None
         self._prepared = False
 
@@ -111,7 +127,7 @@ class RotaryLeading(PositionEncoding):
                 raise ValueError(f"position {positions - 1} lies beyond the {self._tables[0].shape[0]} positions the "
                                  f"rotary table was prepared for")
             rows = max(positions, 2 * (self._tables[0].shape[0] if self._tables is not None else 0))
-            self._tables = _leading_tables(self.dims, self.base, self.env.device, rows, self.factor)
+            self._tables = _leading_tables(self.dims, self.base, self.env.device, rows, self.factor, self.wave)
         return self._tables
 
     def prepare(self, max_positions):

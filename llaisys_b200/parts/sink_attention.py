@@ -9,13 +9,17 @@ from .base import KVNeed, Mixer, TensorDecl, build_part, register_part
 
 @register_part("mixer", "windowed_sink_attention")
 class WindowedSinkAttention(Mixer):
-    """Causal grouped-query attention over the paged cache with six options the plain one does not have:
+    """Causal grouped-query attention over the paged cache with options the plain one does not have:
 
       * keys and queries of `key_dim` elements, values (and the heads' outputs) of `value_dim`;
       * a window that keeps a sequence's first keys: the query at position i sees key j <= i when i - j < window or
         j < keep_first (the kept keys stay at their true positions);
       * a sink: the softmax's denominator has one more term e^0 that carries no value, so the weights are
-        e^{s_j} / (1 + sum e^{s_j}) and may sum to less than one;
+        e^{s_j} / (1 + sum e^{s_j}) and may sum to less than one; with sink = "learned" that term is e^{sink_h}, a number
+        per query head (tensor `sink`, [num_heads]) that is neither scaled nor capped;
+      * a cap on the scores (`softcap` c): a scaled score s becomes c tanh(s / c);
+      * an output gate (`gate` "elements"): the concatenated heads are multiplied element by element by sigmoid(Wg h)
+        (tensor `g`, [num_heads * value_dim, hidden_size]) before the output projection;
       * a penalty on distance (`distance_bias`): the score of query position i and key position j loses
         r1[h] ln(1 + r2[h] (i - j)), with two numbers per query head (tensors `r1`, `r2`, [num_heads]);
       * a query temperature (`q_temp` = {coef, every}): the query at position p is multiplied by
@@ -25,7 +29,7 @@ class WindowedSinkAttention(Mixer):
 
     Query heads h of a group of num_heads / num_kv_heads share key/value head h / group.  Scores are (q . k) * scale.
     The position encoding is a part of category "position" that hands out leading_tables() (rotation of a head's
-    first dimensions).  Projections have no bias; q (and k, v when the layer has them) are one matrix.
+    first dimensions).  Projections have no bias; q (and k, v and the gate when the layer has them) are one matrix.
 
     Cache: `cache_window` says what the layer's cache keeps: None (every key: needed when other layers read it, and
     then this layer's window is only a mask) or the window, kept in a ring of pages behind ceil(keep_first / page)
@@ -34,8 +38,8 @@ class WindowedSinkAttention(Mixer):
     otherwise (and in decode) keys and values are appended first and attention reads the cache alone.
 
     params: hidden_size, num_heads, num_kv_heads, key_dim, value_dim, scale, window, keep_first, sink, own_kv,
-    cache_window, position (PartSpec or None: no rotation), distance_bias, q_temp, names (local tensor names of q, k, v, o,
-    r1, r2; default those).
+    cache_window, position (PartSpec or None: no rotation), distance_bias, q_temp, softcap, gate, names (local tensor names of
+    q, k, v, o, r1, r2, sink, g; default those).
     """
 
     def __init__(self, spec, env):
@@ -52,7 +56,14 @@ class WindowedSinkAttention(Mixer):
         if self.window is not None and self.window <= 0:
             raise ValueError(f"a window holds at least one key, got {self.window}")
         self.keep_first = max(0, int(p.get("keep_first", 0))) if self.window is not None else 0
-        self.sink = bool(p.get("sink", False))
+        self.learned_sink = p.get("sink") == "learned"
+        self.sink = bool(p.get("sink", False)) and not self.learned_sink
+        self.softcap = float(p.get("softcap") or 0.0)
+        if self.softcap < 0:
+            raise ValueError(f"a cap on the scores is positive, got {self.softcap}")
+        if p.get("gate") not in (None, "elements"):
+            raise ValueError(f"the output gate is per 'elements' or absent, got {p.get('gate')!r}")
+        self.gated = p.get("gate") is not None
         self.own_kv = bool(p.get("own_kv", True))
         self.cache_window = p.get("cache_window")
         if self.cache_window is not None and (self.window is None or self.cache_window < self.window):
@@ -61,14 +72,14 @@ class WindowedSinkAttention(Mixer):
         if self.position is not None and not hasattr(self.position, "leading_tables"):
             raise ValueError("this mixer takes a position encoding that rotates a head's leading dimensions")
         self.rot = self.position.dims if self.position is not None else 0
-        self.names = dict({"q": "q", "k": "k", "v": "v", "o": "o", "r1": "r1", "r2": "r2"}, **(p.get("names") or {}))
+        self.names = dict({"q": "q", "k": "k", "v": "v", "o": "o", "r1": "r1", "r2": "r2", "sink": "sink", "g": "g"}, **(p.get("names") or {}))
         self.distance_bias = bool(p.get("distance_bias", False))
         self.q_temp = None
         if p.get("q_temp"):
             self.q_temp = (float(p["q_temp"]["coef"]), int(p["q_temp"]["every"]))
             if self.q_temp[1] <= 0:
                 raise ValueError(f"the query temperature's period must be positive, got {self.q_temp[1]}")
-        self.w_in = self.w_o = self.r1 = self.r2 = None
+        self.w_in = self.w_o = self.r1 = self.r2 = self.sink_logits = None
 
     capturable = True
 
@@ -85,6 +96,10 @@ class WindowedSinkAttention(Mixer):
         if self.own_kv:
             t[n["k"]] = TensorDecl((self.nkvh * self.dk, self.hidden))
             t[n["v"]] = TensorDecl((self.nkvh * self.dv, self.hidden))
+        if self.learned_sink:
+            t[n["sink"]] = TensorDecl((self.nh,), use="vector")
+        if self.gated:
+            t[n["g"]] = TensorDecl((self.nh * self.dv, self.hidden))
         if self.distance_bias:
             t[n["r1"]] = TensorDecl((self.nh,), init="one_plus_normal", use="vector")
             t[n["r2"]] = TensorDecl((self.nh,), init="one_plus_normal", use="vector")
@@ -92,12 +107,15 @@ class WindowedSinkAttention(Mixer):
 
     def load(self, tensors):
         n = self.names
-        ts = [tensors[n["q"]]] + ([tensors[n["k"]], tensors[n["v"]]] if self.own_kv else [])
+        ts = [tensors[n["q"]]] + ([tensors[n["k"]], tensors[n["v"]]] if self.own_kv else []) + ([tensors[n["g"]]] if self.gated else [])
         dt = ts[0].dtype
         for t in ts[1:]:
             dt = torch.promote_types(dt, t.dtype)
         self.w_in = torch.cat([t.to(dt) for t in ts], dim=0).contiguous()
         self.w_o = tensors[n["o"]].contiguous()
+        self.gate_off = self.w_in.shape[0] - self.nh * self.dv              # the gate's columns, when there is one
+        if self.learned_sink:
+            self.sink_logits = tensors[n["sink"]].float().contiguous()
         if self.distance_bias:
             self.r1, self.r2 = tensors[n["r1"]].float().contiguous(), tensors[n["r2"]].float().contiguous()
 
@@ -121,11 +139,17 @@ class WindowedSinkAttention(Mixer):
         return max(1, splits)
 
     def _attend(self, x, ctx, call):
-        """Projections, rotation, cache append and attention: [T, nh * value_dim], before the output projection."""
+        """Projections, rotation, cache append, attention and gate: [T, nh * value_dim], before the output projection."""
+        proj = kernels.linear(x, self.w_in)
+        heads = self._heads(proj, ctx, call)
+        if self.gated:
+            kernels.head_gate_(heads, proj[:, self.gate_off:], self.nh * self.dv)
+        return heads
+
+    def _heads(self, proj, ctx, call):
         kv = ctx.kv(call)
         if kv.writable != self.own_kv:
             raise ValueError("a layer with key/value projections keeps its own cache; one without reads another layer's")
-        proj = kernels.linear(x, self.w_in)
         nkv_here = self.nkvh if self.own_kv else 0
         tables = self.position.leading_tables(ctx.max_position + 1) if self.position is not None else None
         cos, sin = tables if tables is not None else (None, None)
@@ -134,6 +158,7 @@ class WindowedSinkAttention(Mixer):
             append = dict(tok_seq=ctx.tok_seq, seq_start=ctx.seq_start, seq_len_before=ctx.seq_len_before, kpool=kv.k,
                           vpool=kv.v, page_table=kv.page_table, ring=kv.ring, pinned=kv.pinned)
         extras = kernels.AttnExtras(value_dim=self.dv, keep_first=self.keep_first, pinned=kv.pinned, sink=self.sink,
+                                    sink_logits=self.sink_logits, softcap=self.softcap,
                                     dist_bias=(self.r1, self.r2) if self.distance_bias else None, q_temp=self.q_temp)
         common = (proj, self.nh, self.nkvh, self.dk, kv.k, kv.v, kv.page_table, kv.ring, ctx.seq_start, ctx.seq_len_before,
                   ctx.n_seqs)
