@@ -611,13 +611,36 @@ def zetalorn_configs(size: str, layers: int):
     return zl, design_configs(size, layers)[0]
 
 
+def bezadra_configs(size: str, layers: int):
+    """(Bezadra config, Nubedra config) of one size: the same width and dense feed-forward, recurrent heads of the same key and
+    value channels, and attention at the heads and head size of the Qwen2 model of that size.  Layers in turn: a
+    recurrent one (delta rule, four taps) and an attention one.  With six layers or more, two of the layers run twice, so
+    that the model has `layers` layer runs from `layers` - 2 layers."""
+    D, H, dn, dr, _, _, _, _, ff, gh, gk, gv, G = NUBEDRA_SIZES[size]
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    kinds = [
+        {"type": "channel_delta", "mlp": dense, "mixer": {"heads": gh, "kv_heads": gh, "dim": gk, "vdim": gv, "conv": 4}},
+        {"type": "attention", "mlp": dense, "mixer": {
+            "heads": H, "kv_heads": G, "dim": dn + dr, "vdim": dn + dr, "scale": (dn + dr) ** -0.5, "softcap": 30.0,
+            "rot": {"dims": dn + dr, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}},
+    ]
+    looped = layers >= 6
+    n = layers - 2 if looped else layers
+    bz = {"architecture": "Bezadra", "vocab": 32768, "width": D, "norm": {"eps": 1e-6}, "embedding": {"scale": float(D) ** 0.5},
+          "logit_scale": 1.0, "layers": [kinds[i % 2] for i in range(n)]}
+    if looped:
+        bz["loop"] = {"start": 2, "stop": 4, "times": 2}
+    return bz, nubedra_configs(size, layers)[0]
+
+
 DESIGNS = {"vumezen": (DESIGN_SIZES, design_configs, "qwen2"), "nubedra": (NUBEDRA_SIZES, nubedra_configs, "qwen2"),
-           "zedirax": (NUBEDRA_SIZES, zedirax_configs, "nubedra"), "zetalorn": (DESIGN_SIZES, zetalorn_configs, "vumezen")}
+           "zedirax": (NUBEDRA_SIZES, zedirax_configs, "nubedra"), "zetalorn": (DESIGN_SIZES, zetalorn_configs, "vumezen"),
+           "bezadra": (NUBEDRA_SIZES, bezadra_configs, "nubedra")}
 
 
 def design_run(args) -> int:
     """Prefill (one step over --tokens tokens) and decode (--batch sequences that hold --tokens tokens each) of the
-    chosen design and of the model beside it (the Qwen2 dense decoder; for zedirax the Nubedra design, for zetalorn the Vumezen design) at equal layer sizes: time per step, tokens a second, and each kernel's
+    chosen design and of the model beside it (the Qwen2 dense decoder; for zedirax and bezadra the Nubedra design, for zetalorn the Vumezen design) at equal layer sizes: time per step, tokens a second, and each kernel's
     share of a step (torch.profiler).  One JSON line per model and phase.  Inputs: the weights of either model are
     larger than L2, and nothing is flushed between steps."""
     import collections
@@ -852,7 +875,7 @@ def main() -> int:
     ap.add_argument("--timeline", choices=["decode", "prefill"], default=None,
                     help="print the per-kernel timeline of a step (torch.profiler, no ncu) instead of measuring")
     ap.add_argument("--design", choices=sorted(DESIGNS), default=None,
-                    help="measure this design beside the Qwen2 dense decoder (zedirax: beside the Nubedra design; zetalorn: beside the Vumezen design) at equal layer sizes "
+                    help="measure this design beside the Qwen2 dense decoder (zedirax, bezadra: beside the Nubedra design; zetalorn: beside the Vumezen design) at equal layer sizes "
                          "(prefill of --tokens tokens, decode at --batch) instead of the benchmark; --size picks among the sizes "
                          "(default: all)")
     ap.add_argument("--size", default=None, help="with --design: comma-separated sizes of " + ", ".join(sorted(DESIGN_SIZES)))

@@ -12,8 +12,7 @@
 //    with a run of its key channels (KPT state values in registers); q, k, a and v of sixteen tokens at a time are
 //    staged in shared memory, the next sixteen being fetched into registers meanwhile; the chunk runs without a branch
 //    and every o_t is completed by shuffles among the lanes of its column, those of a chunk together.
-//  * gla_out: per (token, head) one warp: RMS norm of o over the value channels with a weight shared by the heads,
-//    times silu of the output gate.
+// (The heads' norm and output gate that follow are headout.cu.)
 #include "common.cuh"
 
 constexpr int GLA_THREADS = 128;
@@ -267,40 +266,5 @@ LLB_API int llb_gla_chunk_prefix(float* tmp, float* state, const int* seq_chunk0
     if (B > 65535) return (int)cudaErrorInvalidValue;
     llb_launch(gla_chunk_prefix_kernel, dim3((n_state + 255) / 256, B), dim3(256), 0, stream, tmp, state, seq_chunk0, chunk_len,
                seq_slot, head_decay, per_head, n_state);
-    return llb_status();
-}
-
-// out[t, h * dv + d] = o[t, h, d] / sqrt(mean_d o[t, h, :]^2 + eps) * w[d] * silu(g[t, h * dv + d])      (gate_act 1: sigmoid(g))
-template <typename T, typename TW>
-__global__ void __launch_bounds__(128) gla_out_kernel(const float* __restrict__ o, const T* __restrict__ g, int g_stride,
-                                                      const TW* __restrict__ w, T* __restrict__ out, int rows, int H, int dv,
-                                                      float eps, int gate_act) {
-    const int lane = threadIdx.x & 31;
-    const int r = blockIdx.x * 4 + (threadIdx.x >> 5);       // (token, head)
-    llb_grid_dependency_sync();
-    if (r >= rows) return;
-    const int t = r / H, h = r - t * H;
-    const float* x = o + (size_t)r * dv;
-    float ss = 0.f;
-    for (int d = lane; d < dv; d += 32) ss += x[d] * x[d];
-    ss = warp_sum(ss);
-    const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
-    for (int d = lane; d < dv; d += 32) {
-        float gv = to_f32(g[(size_t)t * g_stride + h * dv + d]);
-        const float sg = 1.0f / (1.0f + expf(-gv));
-        out[(size_t)r * dv + d] = from_f32<T>(x[d] * inv * to_f32(w[d]) * (gate_act == 1 ? sg : gv * sg));
-    }
-}
-
-LLB_API int llb_gla_out(const float* o, const void* g, int g_stride, const void* w, int w_dtype, void* out, int dtype,
-                        int T, int H, int dv, float eps, int gate_act, cudaStream_t stream) {
-    int rows = T * H;
-    if (rows == 0) return 0;
-    LLB_DISPATCH_DTYPE(dtype, TT, {
-        LLB_DISPATCH_DTYPE(w_dtype, TW, {
-            llb_launch(gla_out_kernel<TT, TW>, dim3((rows + 3) / 4), dim3(128), 0, stream, o, (const TT*)g, g_stride,
-                       (const TW*)w, (TT*)out, rows, H, dv, eps, gate_act);
-        });
-    });
     return llb_status();
 }

@@ -8,7 +8,7 @@
 //   layer_norm    out[r] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * weight, v = x[rows ? rows[r] : r]
 //   copy_rows     rows of the stream, converted, into a matrix of another row stride
 //
-// One block (layer_norm of many rows: one warp) per row; a row is read once.
+// One block (layer_norm of many rows: one to four warps) per row; a row is read once.
 #include "common.cuh"
 
 __device__ __forceinline__ float block_sum_256(float v, float* red) {
@@ -166,13 +166,14 @@ template <int TPR>
 __device__ __forceinline__ float row_sum(float v, float* red) {
     v = warp_sum(v);
     if (TPR == 32) return v;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    constexpr int W = TPR / 32;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, first = warp / W * W;
     __syncthreads();
     if (lane == 0) red[warp] = v;
     __syncthreads();
     float s = 0.f;
 #pragma unroll
-    for (int w = 0; w < 8; ++w) s += red[w];
+    for (int w = 0; w < W; ++w) s += red[first + w];
     return s;
 }
 
@@ -182,8 +183,8 @@ __global__ void __launch_bounds__(256) layer_norm_kernel(const float* __restrict
     __shared__ float red[8];
     const int tid = threadIdx.x % TPR, r = blockIdx.x * (256 / TPR) + threadIdx.x / TPR;
     llb_grid_dependency_sync();
-    if (r >= R) return;                                    // (whole warps or whole blocks)
-    const float* src = x + (size_t)(rows ? rows[r] : r) * H;
+    const bool live = r < R;                               // (threads past the end take part in the barriers)
+    const float* src = x + (size_t)(rows ? rows[live ? r : 0] : (live ? r : 0)) * H;
     float4 v[PER];
     float s = 0.f;
 #pragma unroll
@@ -208,7 +209,7 @@ __global__ void __launch_bounds__(256) layer_norm_kernel(const float* __restrict
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
         const int j = (tid + i * TPR) * 4;
-        if (j >= H) continue;
+        if (j >= H || !live) continue;
         const float y[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
         alignas(16) TO o[4];
 #pragma unroll
@@ -240,11 +241,12 @@ static int layer_norm_launch(const float* x, const TW* w, TO* out, const int* ro
     if (H % 4 == 0 && H <= 16384 && !(((uintptr_t)x | (uintptr_t)out) & 15)) {
 #define LLB_LN(TPR, PER) do { llb_launch(layer_norm_kernel<TW, TO, TPR, PER>, dim3((R + 256 / TPR - 1) / (256 / TPR)), dim3(256), 0,     \
                                          stream, x, w, out, rows, R, H, eps); return llb_status(); } while (0)
-        if (R >= 256) {                                    // many rows: a warp per row
+        if (R >= 256) {                                    // many rows: a warp, or four, per row
             if (H <= 512) LLB_LN(32, 4);
-            if (H <= 1024) LLB_LN(32, 8);
-            if (H <= 2048) LLB_LN(32, 16);
-            if (H <= 4096) LLB_LN(32, 32);
+            if (H <= 1024) LLB_LN(128, 2);
+            if (H <= 1536) LLB_LN(128, 3);
+            if (H <= 2048) LLB_LN(128, 4);
+            if (H <= 4096) LLB_LN(128, 8);
         }
         if (H <= 1024) LLB_LN(256, 1);
         if (H <= 2048) LLB_LN(256, 2);

@@ -1,4 +1,4 @@
-"""Python faces of the kernels of the recurrent and the latent mixers (csrc/gla.cu, csrc/delta.cu, csrc/latent.cu, and the CUDA-core
+"""Python faces of the kernels of the recurrent and the latent mixers (csrc/gla.cu, csrc/delta.cu, csrc/headout.cu, csrc/latent.cu, and the CUDA-core
 attention kernel of csrc/attention_simt.cu run over a cache of latent rows)."""
 from __future__ import annotations
 
@@ -9,7 +9,7 @@ from typing import Optional
 import torch
 
 from ..csrc.build import load_module
-from .ops import DT, KernelError, _AttnParams, _attn_lib, _check, _dt, _fn, _need_cuda, _ptr, _sm_count, _stream
+from .ops import DT, KernelError, _AttnParams, _attn_lib, _check, _dt, _fn, _need_cuda, _ptr, _sm_count, _stream, _tc_resources
 
 
 class _GlaParams(ctypes.Structure):
@@ -103,7 +103,7 @@ def gla_out(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, H: int, d
     T = o.shape[0]
     assert o.dtype == torch.float32 and o.is_contiguous() and gate.dtype == out_dtype and gate.stride(1) == 1
     out = torch.empty((T, H * dv), dtype=out_dtype, device=o.device)
-    f = _fn(load_module("gla.cu"), "llb_gla_out", [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
+    f = _fn(load_module("headout.cu"), "llb_gla_out", [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
                                                   c_int, c_float, c_int, c_void_p])
     _check(f(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _dt(weight), _ptr(out), DT[out_dtype], T, H, dv, eps,
              {"silu": 0, "sigmoid": 1}[gate_act], _stream()),
@@ -113,22 +113,22 @@ def gla_out(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, H: int, d
 
 class _DeltaPrepParams(ctypes.Structure):
     _fields_ = [("proj", c_void_p), ("ld", c_int), ("z", c_void_p), ("conv_w", c_void_p), ("a_log", c_void_p), ("conv_state", c_void_p),
-                ("tok_seq", c_void_p), ("seq_start", c_void_p), ("seq_slot", c_void_p), ("out", c_void_p), ("beta", c_void_p),
-                ("T", c_int), ("G", c_int), ("H", c_int), ("dk", c_int), ("dv", c_int), ("taps", c_int), ("q_scale", c_float),
-                ("single", c_int)]
+                ("seq_start", c_void_p), ("seq_slot", c_void_p), ("out", c_void_p), ("beta", c_void_p),
+                ("G", c_int), ("H", c_int), ("dk", c_int), ("dv", c_int), ("taps", c_int), ("q_scale", c_float),
+                ("fast", c_int), ("vec", c_int)]
 
 
 DELTA_MAX_DIM = 256           # key and value channels of a head
 
 
 def delta_prep(proj: torch.Tensor, z: torch.Tensor, conv_w: torch.Tensor, a_log: torch.Tensor, conv_state: Optional[torch.Tensor],
-               G: int, H: int, dk: int, dv: int, q_scale: float, ctx):
+               G: int, H: int, dk: int, dv: int, q_scale: float, ctx, fast: bool = False):
     """What enters the delta rule, from proj [T, >= C + H] (float32; C = 2 G dk + H dv: q, k of G heads and v of H heads, then
     one step-size logit per head) and the decays' logits z [T, H dk] (float32, contiguous, replaced in place by the decays
     exp(-exp(a_log) softplus(z))): (rows [T, C], beta [T, H]) with the short causal convolution (conv_w float32 [taps, C],
     the last row for the current token) and silu applied, every head's q and k made unit vectors (q times q_scale) and
     beta = sigmoid(logit).  conv_state (float32 [slots, (taps - 1) C], oldest input first; None with one tap) holds each
-    sequence's last inputs and is brought up to date."""
+    sequence's last inputs and is brought up to date.  fast: silu by the special-function unit (for the bfloat16 path)."""
     _need_cuda(proj, z, conv_w, a_log, conv_state)
     T = proj.shape[0]
     C, taps = 2 * G * dk + H * dv, conv_w.shape[0]
@@ -139,10 +139,10 @@ def delta_prep(proj: torch.Tensor, z: torch.Tensor, conv_w: torch.Tensor, a_log:
     beta = torch.empty((T, H), dtype=torch.float32, device=proj.device)
     p = _DeltaPrepParams()
     p.proj, p.ld, p.z, p.conv_w, p.a_log, p.conv_state = proj.data_ptr(), proj.stride(0), z.data_ptr(), conv_w.data_ptr(), a_log.data_ptr(), _ptr(conv_state)
-    p.tok_seq, p.seq_start, p.seq_slot, p.out, p.beta = ctx.tok_seq.data_ptr(), ctx.seq_start.data_ptr(), ctx.seq_slot.data_ptr(), out.data_ptr(), beta.data_ptr()
-    p.T, p.G, p.H, p.dk, p.dv, p.taps, p.q_scale, p.single = T, G, H, dk, dv, taps, q_scale, int(ctx.max_new == 1)
-    f = _fn(load_module("delta.cu"), "llb_delta_prep", [_DeltaPrepParams, c_int, c_void_p])
-    _check(f(p, ctx.n_seqs, _stream()), "delta rule (convolution, unit vectors, decays)", 1 if p.single or taps == 1 else 2)
+    p.seq_start, p.seq_slot, p.out, p.beta = ctx.seq_start.data_ptr(), ctx.seq_slot.data_ptr(), out.data_ptr(), beta.data_ptr()
+    p.G, p.H, p.dk, p.dv, p.taps, p.q_scale, p.fast = G, H, dk, dv, taps, q_scale, int(fast)
+    f = _fn(load_module("delta.cu"), "llb_delta_prep", [_DeltaPrepParams, c_int, c_int, c_void_p])
+    _check(f(p, ctx.n_seqs, ctx.max_new, _stream()), "delta rule (convolution, unit vectors, decays)")
     return out, beta
 
 
@@ -153,7 +153,7 @@ class _DeltaScanParams(ctypes.Structure):
 
 class _DeltaChunkParams(ctypes.Structure):
     _fields_ = [("qkv", c_void_p), ("g", c_void_p), ("beta", c_void_p), ("state", c_void_p), ("seq_start", c_void_p), ("seq_slot", c_void_p),
-                ("out", c_void_p), ("rec", c_void_p), ("G", c_int), ("H", c_int), ("dk", c_int), ("dv", c_int), ("np", c_int), ("cb", c_int)]
+                ("out", c_void_p), ("rec", c_void_p), ("err", c_void_p), ("G", c_int), ("H", c_int), ("dk", c_int), ("dv", c_int), ("cb", c_int)]
 
 
 DELTA_CHUNKED_FROM = 32       # steps whose longest sequence brings at least this many tokens run in chunks
@@ -182,9 +182,9 @@ def delta_scan(qkv: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: to
     size = lib.llb_delta_scratch
     size.argtypes, size.restype = [c_int, c_int, c_int, c_int, c_int], ctypes.c_longlong
     rec = torch.empty(int(size(T, n_seqs, H, dk, dv)), dtype=torch.float32, device=qkv.device)
-    p.rec = rec.data_ptr()
-    f = _fn(lib, "llb_delta_chunked", [_DeltaChunkParams, c_int, c_int, c_void_p])
-    _check(f(p, n_seqs, max_new, _stream()), "delta rule (recurrence in chunks)", 2)
+    p.rec, p.err = rec.data_ptr(), _tc_resources(qkv.device)[2].data_ptr()
+    f = _fn(lib, "llb_delta_chunked", [_DeltaChunkParams, c_int, c_int, c_int, c_void_p])
+    _check(f(p, n_seqs, max_new, _sm_count(qkv.device), _stream()), "delta rule (recurrence in chunks)", 2)
     del rec
     return out
 

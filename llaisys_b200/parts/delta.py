@@ -72,7 +72,8 @@ class ChannelDeltaRule(Mixer):
             if tensors[n[second]].shape[1] != tensors[n[first]].shape[0]:
                 raise ValueError(f"the matrices {n[first]} and {n[second]} do not fit: {tuple(tensors[n[first]].shape)} and "
                                  f"{tuple(tensors[n[second]].shape)}")
-        self.w_in = _fuse([tensors[n[k]] for k in ("q", "k", "v", "b")])
+        # (rows of zeros behind beta's keep the product's rows whole 16-byte pieces)
+        self.w_in = _fuse([tensors[n[k]] for k in ("q", "k", "v", "b")] + [tensors[n["b"]].new_zeros((-(self.channels + self.nh) % 8, self.hidden))])
         self.conv = torch.cat([tensors[n[k] + self.conv_suffix].float() for k in ("q", "k", "v")], dim=0).t().contiguous()      # [taps, channels]
         # the second matrices read whole 16-byte pieces of the bottlenecks' rows: each bottleneck is padded with zero rows
         pad = lambda t, r: torch.cat([t, t.new_zeros((-r % 8, t.shape[1]))], dim=0)
@@ -92,7 +93,7 @@ class ChannelDeltaRule(Mixer):
         z = kernels.linear(low[:, :A], self.w_a2, self.b_a2, out_dtype=torch.float32)
         gate = kernels.linear(low[:, A:], self.w_g2)
         qkv, beta = kernels.delta_prep(proj, z, self.conv, self.a_log, ctx.state(call + 1) if self.taps > 1 else None, self.nkh, self.nh,
-                                       self.dk, self.dv, self.q_scale, ctx)
+                                       self.dk, self.dv, self.q_scale, ctx, fast=x.dtype == torch.bfloat16)
         chunked = x.dtype == torch.bfloat16 and ctx.max_new >= kernels.mixers.DELTA_CHUNKED_FROM
         o = kernels.delta_scan(qkv, z, beta, ctx.state(call), ctx.seq_start, ctx.seq_slot, ctx.n_seqs, ctx.max_new, self.nkh, self.nh,
                                self.dk, self.dv, chunked=chunked)
