@@ -102,6 +102,25 @@ __device__ __forceinline__ float llb_tanh_fast(float x) {
     return fmaf(-2.0f, r, 1.0f);
 }
 
+// How a fused gate/up product combines a gate value g and an up value u:
+//     g' = min(g, limit), u' = clamp(u, -limit, limit), out = (u' + plus) * g' / (1 + e^(-alpha g'))
+// The default is SwiGLU, u * g / (1 + e^-g).
+struct GluForm {
+    float limit = __builtin_huge_valf();
+    float alpha = 1.0f;
+    float plus = 0.0f;
+};
+// by the special-function unit, without the steps that rescale subnormal arguments and results: the result is rounded to
+// bfloat16, and those decide nothing in it (e^-g below 1e-38 adds nothing to 1)
+__device__ __forceinline__ float glu_form(float g, float u, const GluForm& f) {
+    g = fminf(g, f.limit);
+    u = fminf(fmaxf(u, -f.limit), f.limit) + f.plus;
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-1.4426950408889634f * f.alpha * g));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return u * g * r;
+}
+
 static inline int llb_status() { return (int)cudaGetLastError(); }
 
 // ---- programmatic dependent launch

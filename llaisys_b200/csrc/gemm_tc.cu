@@ -58,6 +58,7 @@ struct GemmArgs {
     float* scratch;        // [tiles][splits][accs][BN][BM] float32
     int* counters;         // [tiles], zero between launches
     int* err;
+    GluForm glu = {};      // DUAL: how gate and up combine
 };
 
 template <int BN, int STAGES, bool DUAL>
@@ -244,7 +245,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
     };
     auto finish_at = [&](float acc0, float acc1, int j, int row, float bias_v) {
         float v = acc0;
-        if (DUAL) v = acc1 * __fdividef(acc0, 1.0f + __expf(-acc0));
+        if (DUAL) v = glu_form(acc0, acc1, g.glu);
         v += bias_v;
         size_t o = (size_t)(n0 + j) * g.ldy + row;
         if (g.y_dtype == LLB_F32) ((float*)g.Y)[o] = v;
@@ -294,7 +295,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                 for (int j = 0; j < 16; ++j) {
                     float v = v0[j];
-                    if (DUAL) v = v1[j] * __fdividef(v, 1.0f + __expf(-v));      // fast division: the result is rounded to bfloat16
+                    if (DUAL) v = glu_form(v, v1[j], g.glu);
                     stg[(c + j) * BM + tid] = __float2bfloat16_rn(v + bias_v);
                 }
             }
@@ -657,7 +658,7 @@ gateup_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
                 const float gate = v[j], up = xch[(c + j) * HALF + tid];
-                stg[(c + j) * HALF + tid] = __float2bfloat16_rn(up * __fdividef(gate, 1.0f + __expf(-gate)));   // fast division: the result is rounded to bfloat16
+                stg[(c + j) * HALF + tid] = __float2bfloat16_rn(glu_form(gate, up, g.glu));
             }
         }
     }
@@ -709,10 +710,12 @@ static long long llb_gemm_tc_scratch_elems(int T, int N, int bn, int splits, int
 // bn: tokens per tile (16, 32, 64, 128, 256).  cluster: reduce the splits through a thread-block cluster where
 // that applies (splits 2, 4, 8 or 16 and bn <= 128), else through `scratch`.  Requirements: K and ldx multiples of 8, X and W 16-byte
 // aligned.  Returns 0, a cudaError, or cudaErrorInvalidValue for a shape it does not take.
-LLB_API int llb_gemm_tc(const void* X, const void* W, const void* bias, int bias_dtype, void* Y, int y_dtype,
-                        int T, int N, int K, int ldx, int ldy, int bn, int splits, int cluster, int dual_offset,
+// dual_offset > 0: gate and up combine as SwiGLU (llb_gemm_tc) or as the form given by limit, alpha and plus
+// (llb_gemm_tc_glu; see GluForm).
+static int gemm_tc_run(const void* X, const void* W, const void* bias, int bias_dtype, void* Y, int y_dtype,
+                       int T, int N, int K, int ldx, int ldy, int bn, int splits, int cluster, int dual_offset,
                         float* scratch, long long scratch_elems, int* counters, int n_counters, int* err,
-                        cudaStream_t stream) {
+                       const GluForm& glu, cudaStream_t stream) {
     if (T <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ldx % 8 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
     if (y_dtype != LLB_F32 && y_dtype != LLB_BF16) return (int)cudaErrorInvalidValue;
@@ -740,7 +743,7 @@ LLB_API int llb_gemm_tc(const void* X, const void* W, const void* bias, int bias
     if (rc) return rc;
     rc = llb_tma::bf16_map_64(X, T, K, ldx, bn, &mx);
     if (rc) return rc;
-    GemmArgs g{bias, bias_dtype, Y, y_dtype, T, N, K, ldy, dual_offset, splits, cluster, scratch, counters, err};
+    GemmArgs g{bias, bias_dtype, Y, y_dtype, T, N, K, ldy, dual_offset, splits, cluster, scratch, counters, err, glu};
 #define LLB_TC(BN_, ST_, STD_) \
     case BN_: return dual ? launch<BN_, STD_, true>(mw, mx, g, grid, stream) : launch<BN_, ST_, false>(mw, mx, g, grid, stream)
     switch (bn) {
@@ -754,12 +757,26 @@ LLB_API int llb_gemm_tc(const void* X, const void* W, const void* bias, int bias
 #undef LLB_TC
 }
 
+LLB_API int llb_gemm_tc(const void* X, const void* W, const void* bias, int bias_dtype, void* Y, int y_dtype,
+                        int T, int N, int K, int ldx, int ldy, int bn, int splits, int cluster, int dual_offset,
+                         float* scratch, long long scratch_elems, int* counters, int n_counters, int* err,
+                         cudaStream_t stream) {
+    return gemm_tc_run(X, W, bias, bias_dtype, Y, y_dtype, T, N, K, ldx, ldy, bn, splits, cluster, dual_offset, scratch, scratch_elems, counters, n_counters, err, GluForm{}, stream);
+}
+
+LLB_API int llb_gemm_tc_glu(const void* X, const void* W, const void* bias, int bias_dtype, void* Y, int y_dtype,
+                            int T, int N, int K, int ldx, int ldy, int bn, int splits, int cluster, int dual_offset,
+                             float* scratch, long long scratch_elems, int* counters, int n_counters, int* err, float limit, float alpha,
+                            float plus, cudaStream_t stream) {
+    return gemm_tc_run(X, W, bias, bias_dtype, Y, y_dtype, T, N, K, ldx, ldy, bn, splits, cluster, dual_offset, scratch, scratch_elems, counters, n_counters, err, GluForm{limit, alpha, plus}, stream);
+}
+
 // The fused gate/up product for 17 to 64 tokens with a block per 64 outputs (gateup_tc_kernel): X [T, K] bf16 with
 // row stride ldx, W [2 I, K] bf16 dense (gate rows first), Y [T, I] bf16 with row stride ldy.  bn: tokens per tile
 // (32 or 64; with larger tiles the kernel above was measured as fast or faster).  K, ldx, ldy and I multiples of 8,
 // all three 16-byte aligned; cudaErrorInvalidValue otherwise.
 LLB_API int llb_gemm_tc_gateup(const void* X, const void* W, void* Y, int T, int I, int K, int ldx, int ldy, int bn,
-                               int* err, cudaStream_t stream) {
+                               float limit, float alpha, float plus, int* err, cudaStream_t stream) {
     if (T <= 0 || I <= 0) return 0;
     if (K <= 0 || K % 8 || ldx % 8 || ldy % 8 || I % 8 || (((uintptr_t)X | (uintptr_t)W | (uintptr_t)Y) & 15))
         return (int)cudaErrorInvalidValue;
@@ -770,7 +787,7 @@ LLB_API int llb_gemm_tc_gateup(const void* X, const void* W, void* Y, int T, int
     if (rc) return rc;
     rc = llb_tma::bf16_map_64(X, T, K, ldx, bn, &mx);
     if (rc) return rc;
-    GemmArgs g{nullptr, 0, Y, LLB_BF16, T, 2 * I, K, ldy, I, 1, 0, nullptr, nullptr, err};
+    GemmArgs g{nullptr, 0, Y, LLB_BF16, T, 2 * I, K, ldy, I, 1, 0, nullptr, nullptr, err, GluForm{limit, alpha, plus}};
     switch (bn) {
         case 32: return launch_gateup<32, 8>(mw, mx, g, grid, stream);        // 160 KB of ring
         case 64: return launch_gateup<64, 8>(mw, mx, g, grid, stream);        // 192 KB (with 96 KB, two blocks to an SM: slower)

@@ -155,12 +155,6 @@ __device__ __forceinline__ void tmem_ld_cols_nowait(uint32_t taddr, uint32_t* r)
                  : "r"(taddr) : "memory");
 }
 
-// The two special-function results of a SwiGLU output as single instructions: without .ftz each of them comes with
-// a few more that rescale subnormal arguments and results, which decide nothing here (exp(-gate) below 1e-38 adds
-// nothing to 1, and a quotient below 1e-38 is rounded to a bfloat16 zero either way).
-__device__ __forceinline__ float ex2_ftz(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
-__device__ __forceinline__ float rcp_ftz(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
-
 struct Gemm2Args {
     const void* bias;      // [rows_out] or null
     int bias_dtype;
@@ -171,6 +165,7 @@ struct Gemm2Args {
     int tok_tiles, n_tiles, n_pairs;
     int* err;
     int ksplit, chunk_kb;  // INTO: K ranges per tile and k-blocks per range (1 and all of them otherwise)
+    GluForm glu = {};      // DUAL: how gate and up combine
 };
 
 // The loads issued so far have arrived.  The registers pass through the statement so that no use of them is
@@ -435,8 +430,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                 }
                 if (DUAL == 2) {
 #pragma unroll
-                    for (int j = 0; j < COLS; ++j)                                  // up * gate / (1 + exp(-gate))
-                        v0[j] = v1[j] * v0[j] * rcp_ftz(1.0f + ex2_ftz(-1.4426950408889634f * v0[j]));
+                    for (int j = 0; j < COLS; ++j) v0[j] = glu_form(v0[j], v1[j], g.glu);
                 } else if (DUAL == 1) {
                     // The up warp writes buffer chunk_i & 1 and meets the gate warp at their barrier; it writes that buffer
                     // again two chunks on, behind the next chunk's barrier, which the gate warp reaches after these reads.
@@ -449,8 +443,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                     }
                     asm volatile("bar.sync %0, 64;" ::"r"(2 + xpair) : "memory");
 #pragma unroll
-                    for (int j = 0; j < COLS; ++j)                                  // up * gate / (1 + exp(-gate))
-                        v0[j] = xb[j * 32 + lane] * v0[j] * rcp_ftz(1.0f + ex2_ftz(-1.4426950408889634f * v0[j]));
+                    for (int j = 0; j < COLS; ++j) v0[j] = glu_form(v0[j], xb[j * 32 + lane], g.glu);
                 } else {
 #pragma unroll
                     for (int j = 0; j < COLS; ++j) v0[j] += bias_v;
@@ -543,7 +536,8 @@ LLB_DEFINE_SET_STAMPS
 // bf16; bias [N] or null.  max_pairs: how many CTA pairs may run at once (SMs / 2).  Returns
 // cudaErrorInvalidValue for what this kernel does not take (the caller then uses the one-CTA kernel).
 LLB_API int llb_gemm_tc2(const void* X, const void* W, const void* bias, int bias_dtype, void* Y, int T, int N, int K,
-                         int ldx, int ldy, int dual_offset, int max_pairs, int* err, cudaStream_t stream) {
+                         int ldx, int ldy, int dual_offset, float limit, float alpha, float plus, int max_pairs, int* err,
+                         cudaStream_t stream) {
     if (T == 0 || N == 0) return 0;
     const int dual = dual_offset > 0;
     const int rows_out = dual ? dual_offset : N;
@@ -566,6 +560,7 @@ LLB_API int llb_gemm_tc2(const void* X, const void* W, const void* bias, int bia
     g.n_tiles = (int)tiles;
     g.n_pairs = (int)(tiles < max_pairs ? tiles : max_pairs);
     g.err = err;
+    g.glu = GluForm{limit, alpha, plus};
     g.ksplit = 1;
     g.chunk_kb = (K + BK - 1) / BK;
     CUtensorMap mw, mx;

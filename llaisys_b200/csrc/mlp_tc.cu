@@ -148,6 +148,7 @@ struct MlpArgs {
     int n_mt;              // ceil(H / 128): output row tiles of the down projection
     int tmem_cols;         // power of two >= 2 BN + n_mt BN
     int* err;
+    GluForm glu = {};      // how gate and up combine
 };
 
 template <int BN, int STAGES>
@@ -374,13 +375,13 @@ mlp_fused_kernel(const __grid_constant__ CUtensorMap map_gate, const __grid_cons
                     ok = false;
                     break;
                 }
-                // act[n][col] = up * gate / (1 + exp(-gate)), bfloat16, into the swizzled K-major tile: row n (token) is
+                // act[n][col] = the gated activation (GluForm), bfloat16, into the swizzled K-major tile: row n (token) is
                 // 128 bytes; its 16-byte piece col / 8 sits at piece (col / 8) ^ (n % 8); groups of 8 rows are 1024 bytes
                 uint8_t* act = gen_base + S::ACT_OFFSET + b * S::ACT_BYTES;
 #pragma unroll
                 for (int n = 0; n < BN; ++n) {
                     const float gate = v[n], up = exch[col * BN + n];
-                    const float a = up * __fdividef(gate, 1.0f + __expf(-gate));
+                    const float a = glu_form(gate, up, g.glu);
                     const int off = (n >> 3) * 1024 + (n & 7) * 128 + ((((col >> 3) ^ (n & 7)) & 7) << 4) + (col & 7) * 2;
                     *reinterpret_cast<bf16*>(act + off) = __float2bfloat16_rn(a);
                 }
@@ -485,12 +486,12 @@ LLB_API int llb_mlp_fused_ok(int T, int H, int I) {
 }
 
 // X [T, H] bf16 (row stride ldx), Wgu [2 I, H] bf16 dense (gate rows first), Wd [H, I] bf16 dense;
-// residual [T, H] float32 dense += the feed-forward of X.  blocks: the most blocks to launch (the SM count).
+// residual [T, H] float32 dense += the feed-forward of X, gate and up combined as limit, alpha and plus say (GluForm).  blocks: the most blocks to launch (the SM count).
 // stages: depth of the TMA ring (4, 5, 6, 8, and 10 for up to 16 tokens; 0 chooses).
 LLB_DEFINE_SET_STAMPS
 
 LLB_API int llb_mlp_fused(const void* X, int ldx, const void* Wgu, const void* Wd, float* residual, int T, int H, int I,
-                          int blocks, int stages, int* err, cudaStream_t stream) {
+                          int blocks, int stages, float limit, float alpha, float plus, int* err, cudaStream_t stream) {
     if (!llb_mlp_fused_ok(T, H, I) || ldx % 8 || blocks <= 0) return (int)cudaErrorInvalidValue;
     if (((uintptr_t)X | (uintptr_t)Wgu | (uintptr_t)Wd | (uintptr_t)residual) & 15) return (int)cudaErrorInvalidValue;
     const int bn = T <= 16 ? 16 : 32;
@@ -503,6 +504,7 @@ LLB_API int llb_mlp_fused(const void* X, int ldx, const void* Wgu, const void* W
     while (pow2 < cols) pow2 *= 2;
     g.tmem_cols = pow2;
     g.err = err;
+    g.glu = GluForm{limit, alpha, plus};
     CUtensorMap mg, mu, mx, md, mr;
     int rc = llb_tma::bf16_map_64(Wgu, I, H, H, SLICE, &mg);
     if (rc) return rc;

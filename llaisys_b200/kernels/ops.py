@@ -523,25 +523,37 @@ def _pair_ok(out, rows_out) -> bool:
     return out.dtype == torch.bfloat16 and rows_out % 8 == 0 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
 
 
-def _gemm_tc_pair(x, weight, bias, out, dual_offset=0):
+@dataclass(frozen=True)
+class GluForm:
+    """How a fused gate/up product combines a gate value g and an up value u: g' = min(g, limit), u' = clamp(u, -limit, limit),
+    (u' + plus) g' / (1 + e^(-alpha g')).  The default is SwiGLU."""
+    limit: float = float("inf")
+    alpha: float = 1.0
+    plus: float = 0.0
+
+
+SWIGLU = GluForm()
+
+
+def _gemm_tc_pair(x, weight, bias, out, dual_offset=0, glu=SWIGLU):
     """The product on pairs of SMs (csrc/gemm_tc2.cu): persistent, for many tokens, bfloat16 output."""
     M, K = x.shape
     N = weight.shape[0]
     err = _tc_resources(x.device)[2]
     f = _fn(_stamped("gemm_tc2.cu"), "llb_gemm_tc2",
-            [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+            [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p, c_void_p])
     _check(f(_ptr(x), _ptr(weight), _ptr(bias), _dt(bias) if bias is not None else 0, _ptr(out), M, N, K,
-             x.stride(0), out.stride(0), dual_offset, _sm_count(x.device) // 2, _ptr(err), _stream()),
+             x.stride(0), out.stride(0), dual_offset, glu.limit, glu.alpha, glu.plus, _sm_count(x.device) // 2, _ptr(err), _stream()),
            "linear (tensor cores, paired SMs)")
 
 
-def _gemm_tc(x, weight, bias, out, dual_offset=0, plan=None):
+def _gemm_tc(x, weight, bias, out, dual_offset=0, plan=None, glu=SWIGLU):
     M, K = x.shape
     N = weight.shape[0]
     if plan is None and M > 256 and _pair_ok(out, dual_offset or N):
         plan = ("pair",)
     if plan is not None and plan[0] == "pair":
-        return _gemm_tc_pair(x, weight, bias, out, dual_offset)
+        return _gemm_tc_pair(x, weight, bias, out, dual_offset, glu)
     scratch, counters, err = _tc_resources(x.device)
     # gate/up for 17 to 64 tokens: a block per 64 outputs (gate and up rows side by side in one accumulator), twice as
     # many blocks as with a tile of 128 gate rows, which without a K split leaves half of the SMs idle at these sizes
@@ -551,8 +563,9 @@ def _gemm_tc(x, weight, bias, out, dual_offset=0, plan=None):
     if side_by_side and dual_offset and bias is None and _pair_ok(out, dual_offset):
         bn = plan[1] if plan is not None else (32 if M <= 32 else 64)
         f = _fn(_stamped("gemm_tc.cu"), "llb_gemm_tc_gateup",
-                [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
-        _check(f(_ptr(x), _ptr(weight), _ptr(out), M, dual_offset, K, x.stride(0), out.stride(0), bn, _ptr(err), _stream()),
+                [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_void_p])
+        _check(f(_ptr(x), _ptr(weight), _ptr(out), M, dual_offset, K, x.stride(0), out.stride(0), bn, glu.limit, glu.alpha, glu.plus,
+                 _ptr(err), _stream()),
                "gate/up (tensor cores, rows side by side)")
         return
     if side_by_side:
@@ -560,12 +573,12 @@ def _gemm_tc(x, weight, bias, out, dual_offset=0, plan=None):
     plan = plan or tc_plan(M, dual_offset or N, K, _sm_count(x.device), bool(dual_offset))
     bn, splits = plan[0], plan[1]
     cluster = plan[2] if len(plan) > 2 else 1            # (bn, splits, 0) forces the reduction through scratch
-    f = _fn(_stamped("gemm_tc.cu"), "llb_gemm_tc",
+    f = _fn(_stamped("gemm_tc.cu"), "llb_gemm_tc_glu",
             [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p])
+             c_int, c_int, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_float, c_float, c_float, c_void_p])
     _check(f(_ptr(x), _ptr(weight), _ptr(bias), _dt(bias) if bias is not None else 0, _ptr(out), _dt(out),
              M, N, K, x.stride(0), out.stride(0), bn, splits, cluster, dual_offset, _ptr(scratch), scratch.numel(),
-             _ptr(counters), counters.numel(), _ptr(err), _stream()), "linear (tensor cores)")
+             _ptr(counters), counters.numel(), _ptr(err), glu.limit, glu.alpha, glu.plus, _stream()), "linear (tensor cores)")
 
 
 def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
@@ -637,16 +650,20 @@ def linear_into(x: torch.Tensor, weight: torch.Tensor, bias, stream: torch.Tenso
              stream.stride(0), ksplit, _sm_count(x.device) // 2, _ptr(err), _stream()), "linear into the residual stream (tensor cores, paired SMs)")
 
 
-def linear_swiglu(x: torch.Tensor, gate_up: torch.Tensor, plan=None) -> torch.Tensor:
-    """up(x) * silu(gate(x)) for the fused [2I, K] matrix (gate rows first): [M, I].  On the
+def linear_swiglu(x: torch.Tensor, gate_up: torch.Tensor, plan=None, form: GluForm = SWIGLU) -> torch.Tensor:
+    """up(x) * silu(gate(x)), or the combination `form` says, for the fused [2I, K] matrix (gate rows first): [M, I].  On the
     tensor cores the two products share one kernel and the [M, 2I] intermediate is never written."""
     _need_cuda(x, gate_up)
     I = gate_up.shape[0] // 2
     if _tc_ok(x, gate_up, None) and x.shape[0] > 0:
         out = torch.empty((x.shape[0], I), dtype=x.dtype, device=x.device)
-        _gemm_tc(x, gate_up, None, out, dual_offset=I, plan=plan)
+        _gemm_tc(x, gate_up, None, out, dual_offset=I, plan=plan, glu=form)
         return out
-    return swiglu(linear(x, gate_up))
+    if form == SWIGLU:
+        return swiglu(linear(x, gate_up))
+    if form.plus != 1.0:
+        raise KernelError(f"gated activation: no kernel of its own combines gate and up as {form}")
+    return glu(linear(x, gate_up), "swish_clamped", limit=form.limit, alpha=form.alpha)
 
 
 FUSED_MLP = __import__("os").environ.get("LLAISYS_FUSED_MLP", "1") != "0"     # tests switch the one-launch feed-forward off to compare
@@ -673,8 +690,9 @@ def mlp_fused_ok(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, res
     return bool(f(T, H, I))
 
 
-def mlp_fused(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, residual: torch.Tensor, stages: int = 0) -> None:
-    """residual [T, H] (float32) += down(up(x) * silu(gate(x))) in one launch; gate_up is [2I, H] with the gate rows
+def mlp_fused(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, residual: torch.Tensor, stages: int = 0,
+              form: GluForm = SWIGLU) -> None:
+    """residual [T, H] (float32) += down(up(x) * silu(gate(x))), or with the combination `form` says, in one launch; gate_up is [2I, H] with the gate rows
     first, down [H, I].  See mlp_fused_ok() for what it takes."""
     _need_cuda(x, gate_up, down, residual)
     T, H = x.shape
@@ -682,9 +700,9 @@ def mlp_fused(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, residu
     err = _tc_resources(x.device)[2]
     stages = stages or _MLP_STAGES
     f = _fn(_stamped("mlp_tc.cu", _MLP_DEFINES), "llb_mlp_fused",
-            [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+            [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_void_p])
     _check(f(_ptr(x), x.stride(0), _ptr(gate_up), _ptr(down), _ptr(residual), T, H, I, _sm_count(x.device), stages,
-             _ptr(err), _stream()), "feed-forward (one launch, tensor cores)")
+             form.limit, form.alpha, form.plus, _ptr(err), _stream()), "feed-forward (one launch, tensor cores)")
 
 
 # ------------------------------------------------------------------ attention

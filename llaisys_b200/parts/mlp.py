@@ -54,7 +54,7 @@ class GatedMLP(FeedForward):
     """down(act(gate(x)) * up(x)) with the activation a parameter: "silu", "relu", "gelu_tanh", or "swish_clamped":
     g = min(gate(x), limit), u = clamp(up(x), -limit, limit), down(g sigmoid(alpha g) (u + 1)).  The gate
     and up matrices are kept as one [2I, H] matrix so that one product serves both; the activation and the product of
-    the halves are one pass in float32.  With `bias` every projection has a bias (tensors named after the matrices with
+    the halves are one pass in float32, or (silu and swish_clamped without biases) the epilogue of that product; a few tokens run in one launch.  With `bias` every projection has a bias (tensors named after the matrices with
     `bias_suffix`, default ".b").  The result is returned in float32 (it may be normed or scaled before it joins the
     stream) unless the part is asked to add it to the stream itself.  params: hidden_size, intermediate_size, act, limit and alpha (swish_clamped), bias, bias_suffix, names (local tensor names of gate, up, down)."""
     capturable = True
@@ -70,6 +70,10 @@ class GatedMLP(FeedForward):
             raise ValueError(f"the limit must be positive, got {self.limit}")
         self.names = dict({"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}, **(p.get("names") or {}))
         self.bias, self.bias_suffix = bool(p.get("bias", False)), str(p.get("bias_suffix", ".b"))
+        # what the products' own epilogues can do: no bias, and a sigmoid gate
+        self.form = None
+        if not self.bias and self.act in ("silu", "swish_clamped"):
+            self.form = kernels.GluForm() if self.act == "silu" else kernels.GluForm(self.limit, self.alpha, 1.0)
         self.gate_up = self.down = self.b_gate_up = self.b_down = None
 
     def tensors(self):
@@ -93,8 +97,8 @@ class GatedMLP(FeedForward):
             self.b_down = tensors[self.names["down"] + b].float().contiguous()
 
     def _activated(self, x):
-        if self.act == "silu" and not self.bias:
-            return kernels.linear_swiglu(x, self.gate_up)
+        if self.form is not None:
+            return kernels.linear_swiglu(x, self.gate_up, form=self.form)
         return kernels.glu(kernels.linear(x, self.gate_up, self.b_gate_up), self.act, limit=self.limit, alpha=self.alpha)
 
     def forward(self, x, ctx):
@@ -102,6 +106,9 @@ class GatedMLP(FeedForward):
         return kernels.linear(act, self.down, self.b_down, out_dtype=delta_dtype(act))
 
     def forward_into(self, x, ctx, residual):
+        if self.form is not None and kernels.mlp_fused_ok(x, self.gate_up, self.down, residual):
+            kernels.mlp_fused(x, self.gate_up, self.down, residual, form=self.form)      # a few tokens: one launch
+            return True
         if not kernels.linear_into_ok(x.new_empty((x.shape[0], self.inter)), self.down, self.b_down, residual):
             return False
         kernels.linear_into(self._activated(x), self.down, self.b_down, residual)
