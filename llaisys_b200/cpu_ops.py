@@ -65,14 +65,20 @@ def rope(x: np.ndarray, pos_ids: np.ndarray, theta: float) -> np.ndarray:
     return np.concatenate([a * cos - b * sin, b * cos + a * sin], axis=-1)
 
 
-def rope_leading(x: np.ndarray, pos_ids: np.ndarray, dims: int, base: float) -> np.ndarray:
+def rope_leading(x: np.ndarray, pos_ids: np.ndarray, dims: int, base: float, wave=None) -> np.ndarray:
     """Rotation of the first `dims` dimensions of x [seq, heads, d] in pairs (i, i + dims/2) by the angle
-    p * base^(-2i/dims); the other dimensions pass (not in xsmccc/llaisys)."""
+    p * base^(-2i/dims); the other dimensions pass (not in xsmccc/llaisys).  wave = {factor, low, high, original}: the
+    frequency f of wavelength l = 2 pi / f stays where l < original / high, is divided by factor where l > original / low,
+    and blends linearly in original / l between."""
     x = x.astype(np.float32)
     half = dims // 2
     if half == 0:
         return x
     freq = np.power(float(base), -2.0 * np.arange(half, dtype=np.float64) / dims)
+    if wave:
+        turns = wave["original"] * freq / (2.0 * np.pi)                  # original / wavelength
+        blend = np.clip((turns - wave["low"]) / max(wave["high"] - wave["low"], 1e-300), 0.0, 1.0)
+        freq = freq * (blend + (1.0 - blend) / wave["factor"])
     ang = np.asarray(pos_ids, dtype=np.float64)[:, None] * freq[None, :]
     cos, sin = np.cos(ang)[:, None, :].astype(np.float32), np.sin(ang)[:, None, :].astype(np.float32)
     a, b = x[..., :half], x[..., half:dims]
@@ -95,14 +101,14 @@ def route_top(logits: np.ndarray, bias, top: int, scale: float):
 
 
 def self_attention(q: np.ndarray, k: np.ndarray, v: np.ndarray, scale: float, window=None, keep_first: int = 0,
-                   sink: bool = False, sink_logits=None, dist_bias=None) -> np.ndarray:
+                   sink: bool = False, sink_logits=None, dist_bias=None, softcap: float = 0.0) -> np.ndarray:
     """Causal grouped-query attention of q [qlen, nh, d] over k [kvlen, nkvh, d], v [kvlen, nkvh, dv], the queries being
     the last qlen of the kvlen positions: query i sees keys t <= kvlen - qlen + i; head h reads kv head
     h // (nh / nkvh); softmax with the maximum subtracted (src/ops/self_attention/cpu/self_attention_cpu.cpp:28-112).
     Not in that project: window (a query at position p sees only the keys p - window < t <= p), keep_first (the keys
     t < keep_first stay visible behind the window), sink (one more term e^0 in the denominator, without a value) and
     sink_logits [nh] (that term is e^sink_logits[h] instead), dist_bias = (r1 [nh], r2 [nh]) (the score of query position
-    p and key position t loses r1[h] ln(1 + r2[h] (p - t)))."""
+    p and key position t loses r1[h] ln(1 + r2[h] (p - t))), softcap c > 0 (a scaled score s becomes c tanh(s / c))."""
     qlen, nh, d = q.shape
     kvlen, nkvh, dv = v.shape
     group = nh // nkvh
@@ -115,6 +121,8 @@ def self_attention(q: np.ndarray, k: np.ndarray, v: np.ndarray, scale: float, wi
         visible &= (t[None, :] > cur - window) | (t[None, :] < keep_first)
     for h in range(nh):
         s = (q[:, h, :] @ k[:, h // group, :].T) * np.float32(scale)
+        if softcap:
+            s = np.float32(softcap) * np.tanh(s / np.float32(softcap))
         if dist_bias is not None:
             dist = np.maximum(cur - t[None, :], 0).astype(np.float32)
             s = s - np.float32(dist_bias[0][h]) * np.log1p(np.float32(dist_bias[1][h]) * dist)
@@ -303,4 +311,38 @@ def decayed_linear_recurrence(q: np.ndarray, k: np.ndarray, v: np.ndarray, decay
         state *= a
         state += k[t][:, :, None].astype(np.float32) * v[t][:, None, :].astype(np.float32)
         out[t] = np.einsum("hkv,hk->hv", state, q[t].astype(np.float32))
+    return out
+
+
+def layer_norm(x: np.ndarray, weight: np.ndarray, eps: float) -> np.ndarray:
+    """(x - mean) / sqrt(mean((x - mean)^2) + eps) * w, no bias (not in xsmccc/llaisys)."""
+    x = x.astype(np.float32)
+    d = x - x.mean(axis=-1, keepdims=True, dtype=np.float32)
+    return d / np.sqrt((d * d).mean(axis=-1, keepdims=True, dtype=np.float32) + np.float32(eps)) * weight.astype(np.float32)
+
+
+def causal_conv(x: np.ndarray, weight: np.ndarray, last: np.ndarray):
+    """y[t, c] = sum_j w[c, j] x[t - (taps - 1) + j, c] over x [seq, channels] with the inputs before it in `last`
+    [taps - 1, channels]; returns (y, the inputs the next step needs) (not in xsmccc/llaisys)."""
+    taps, T = weight.shape[1], x.shape[0]
+    rows = np.concatenate([last, x.astype(np.float32)])
+    y = sum(rows[j:j + T] * weight[:, j].astype(np.float32) for j in range(taps))
+    return y.astype(np.float32), rows[rows.shape[0] - (taps - 1):].copy()
+
+
+def unit_rows(x: np.ndarray, eps: float = 1e-6) -> np.ndarray:
+    """x / sqrt(sum(x^2) + eps) over the last axis (not in xsmccc/llaisys)."""
+    x = x.astype(np.float32)
+    return x / np.sqrt((x * x).sum(axis=-1, keepdims=True, dtype=np.float32) + np.float32(eps))
+
+
+def delta_recurrence(q: np.ndarray, k: np.ndarray, v: np.ndarray, g: np.ndarray, beta: np.ndarray, state: np.ndarray) -> np.ndarray:
+    """Per head S <- diag(g_t) S, u = beta_t (v_t - S^T k_t), S <- S + k_t u^T, o_t = S^T q_t over q, k, g [T, H, dk],
+    v [T, H, dv], beta [T, H]; `state` [H, dk, dv] is updated in place (not in xsmccc/llaisys)."""
+    out = np.zeros(v.shape, dtype=np.float32)
+    for t in range(v.shape[0]):
+        state *= g[t][:, :, None]
+        u = beta[t][:, None] * (v[t] - np.einsum("hkv,hk->hv", state, k[t]))
+        state += k[t][:, :, None] * u[:, None, :]
+        out[t] = np.einsum("hkv,hk->hv", state, q[t])
     return out

@@ -18,12 +18,14 @@ import numpy as np
 from .. import cpu_ops
 from ..config.spec import ModelSpec, PartSpec
 
-_KNOWN = {"embedding": {"token_embedding", "scaled_pair_embedding"}, "norm": {"rms_norm"},
+_KNOWN = {"embedding": {"token_embedding", "scaled_pair_embedding"}, "norm": {"rms_norm", "layer_norm"},
           "mixer": {"gqa_attention", "windowed_sink_attention", "gated_linear_attention", "latent_attention", "min_gru",
-                    "differential_attention", "pooled_window_attention", "lightning_attention", "parallel_mixers"},
+                    "differential_attention", "pooled_window_attention", "lightning_attention", "parallel_mixers",
+                    "channel_delta_rule"},
           "ffn": {"swiglu_mlp", "routed_experts", "gated_mlp"},
-          "block": {"pre_norm_residual", "parallel_residual", "sandwich_residual", "depth_averaged_residual", "gated_residual"},
-          "head": {"lm_head"}, "reentry": {"embedding_and_offset"},
+          "block": {"pre_norm_residual", "parallel_residual", "sandwich_residual", "depth_averaged_residual", "gated_residual",
+                    "shared_norm_parallel"},
+          "head": {"lm_head"}, "reentry": {"embedding_and_offset", "embedding_projection"},
           "position": {"rope_half_split", "rope_leading", "rope_interleaved"}}
 
 
@@ -68,6 +70,8 @@ class CpuModel:
     # ---- parts
     def _norm(self, p: PartSpec, x):
         w = self.w[p.tensor_name(p.params.get("tensor", "weight"))]
+        if p.kind == "layer_norm":
+            return cpu_ops.layer_norm(x, w, p.params["eps"])
         if p.params.get("offset"):
             w = w.astype(np.float32) + np.float32(p.params["offset"])       # stored as the distance from the offset
         return cpu_ops.rms_norm(x, w, p.params["eps"])
@@ -89,6 +93,29 @@ class CpuModel:
         o = cpu_ops.rms_norm(o, w("norm"), a["eps"]).reshape(T, H * dv)
         g = cpu_ops.linear(x, w("g"))
         return cpu_ops.linear(o * (g / (np.float32(1) + np.exp(-g))), w("o"))
+
+    def _delta_rule(self, p: PartSpec, x, store: dict, key):
+        a = p.params
+        H, G, dk, dv, taps = a["num_heads"], a["num_kv_heads"], a["key_dim"], a["value_dim"], a["taps"]
+        n = dict({k: k for k in ("q", "k", "v", "b", "A_log", "norm", "a1", "a2", "dt_bias", "g1", "g2", "o")}, **(a.get("names") or {}))
+        w = lambda k: self.w[p.tensor_name(n[k])].astype(np.float32)
+        T = x.shape[0]
+        raw = np.concatenate([cpu_ops.linear(x, w(k)) for k in ("q", "k", "v")], axis=1)
+        conv = np.concatenate([self.w[p.tensor_name(n[k] + a.get("conv_suffix", ".conv"))] for k in ("q", "k", "v")]).astype(np.float32)
+        if key not in store:
+            store[key] = (np.zeros((H, dk, dv), dtype=np.float32), np.zeros((taps - 1, raw.shape[1]), dtype=np.float32))
+        S, last = store[key]
+        y, last[:] = cpu_ops.causal_conv(raw, conv, last)
+        y = y * cpu_ops.sigmoid(y)
+        heads = lambda t, m, d: t.reshape(T, m, d)
+        q = cpu_ops.unit_rows(heads(y[:, :G * dk], G, dk)) * np.float32(a.get("query_scale", 1.0))
+        k = cpu_ops.unit_rows(heads(y[:, G * dk:2 * G * dk], G, dk))
+        v = heads(y[:, 2 * G * dk:], H, dv)
+        z = cpu_ops.linear(cpu_ops.linear(x, w("a1")), w("a2"), w("dt_bias")).reshape(T, H, dk)
+        g = np.exp(-np.exp(w("A_log"))[:, None] * (np.maximum(z, 0) + np.log1p(np.exp(-np.abs(z))))).astype(np.float32)
+        o = cpu_ops.delta_recurrence(np.repeat(q, H // G, axis=1), np.repeat(k, H // G, axis=1), v, g, cpu_ops.sigmoid(cpu_ops.linear(x, w("b"))), S)
+        o = cpu_ops.rms_norm(o, w("norm"), a["eps"]).reshape(T, H * dv)
+        return cpu_ops.linear(o * cpu_ops.sigmoid(cpu_ops.linear(cpu_ops.linear(x, w("g1")), w("g2"))), w("o"))
 
     def _min_gru(self, p: PartSpec, x, store: dict, key):
         a = p.params
@@ -146,7 +173,11 @@ class CpuModel:
         sfx = p.params.get("bias_suffix", ".b")
         b = (lambda k: self.w[p.tensor_name(n[k] + sfx)]) if p.params.get("bias") else (lambda k: None)
         g, u = cpu_ops.linear(x, self.w[p.tensor_name(n["gate"])], b("gate")), cpu_ops.linear(x, self.w[p.tensor_name(n["up"])], b("up"))
-        return cpu_ops.linear(cpu_ops.glu(g, u, p.params.get("act", "silu")), self.w[p.tensor_name(n["down"])], b("down"))
+        if p.params.get("act") == "swish_clamped":
+            act = cpu_ops.swish_clamped(g, u, p.params.get("limit", float("inf")), p.params.get("alpha", 1.0))
+        else:
+            act = cpu_ops.glu(g, u, p.params.get("act", "silu"))
+        return cpu_ops.linear(act, self.w[p.tensor_name(n["down"])], b("down"))
 
     # ---- mixers with normed heads, blocks of keys, two score maps, a constant-decay recurrence
     def _normed_rows(self, p: PartSpec, x, positions, maps: int):
@@ -244,6 +275,8 @@ class CpuModel:
         kind = sub.part.kind
         if kind in ("differential_attention", "pooled_window_attention", "lightning_attention", "parallel_mixers"):
             return self._mixer_of(sub.part, h, positions, store, m)
+        if kind == "channel_delta_rule":
+            return self._delta_rule(sub.part, h, store, m)
         if kind == "gated_linear_attention":
             return self._gla(sub.part, h, store, m)
         if kind == "min_gru":
@@ -280,10 +313,12 @@ class CpuModel:
     def _sink_attention(self, p: PartSpec, x, positions, store: dict, key, owner):
         a = p.params
         nh, nkvh, dk, dv = a["num_heads"], a["num_kv_heads"], a["key_dim"], a["value_dim"]
-        n = dict({"q": "q", "k": "k", "v": "v", "o": "o", "r1": "r1", "r2": "r2"}, **(a.get("names") or {}))
+        n = dict({"q": "q", "k": "k", "v": "v", "o": "o", "r1": "r1", "r2": "r2", "sink": "sink", "g": "g"}, **(a.get("names") or {}))
         T = x.shape[0]
         pos = a.get("position")
-        rot = (lambda t: cpu_ops.rope_leading(t, positions, pos.params["dims"], pos.params["base"])) if pos is not None else (lambda t: t)
+        rot = lambda t: t
+        if pos is not None:
+            rot = lambda t: cpu_ops.rope_leading(t, positions, pos.params["dims"], pos.params["base"], pos.params.get("wave"))
         q = rot(cpu_ops.linear(x, self.w[p.tensor_name(n["q"])]).reshape(T, nh, dk))
         if a.get("q_temp"):
             q = q * cpu_ops.query_temperature(positions, a["q_temp"]["coef"], a["q_temp"]["every"])[:, None, None]
@@ -296,7 +331,11 @@ class CpuModel:
             ks, vs = store[key]
         else:
             ks, vs = owner[key]
-        o = cpu_ops.self_attention(q, ks, vs, a["scale"], a.get("window"), a.get("keep_first", 0), bool(a.get("sink")), dist_bias=bias)
+        o = cpu_ops.self_attention(q, ks, vs, a["scale"], a.get("window"), a.get("keep_first", 0), bool(a.get("sink")), dist_bias=bias,
+                                   sink_logits=self.w[p.tensor_name(n["sink"])] if a.get("sink") == "learned" else None,
+                                   softcap=a.get("softcap") or 0.0)
+        if a.get("gate"):
+            o = o * cpu_ops.sigmoid(cpu_ops.linear(x, self.w[p.tensor_name(n["g"])])).reshape(o.shape)
         return cpu_ops.linear(o.reshape(T, nh * dv), self.w[p.tensor_name(n["o"])])
 
     def _routed(self, p: PartSpec, x):
@@ -369,17 +408,21 @@ class CpuModel:
             if call.opens_pass is not None:
                 re = self.spec.reentry
                 offsets = self.w[re.tensor_name(re.params.get("tensor", "offset"))].astype(np.float32)
-                if call.opens_pass > 0:
+                if re.kind == "embedding_projection":              # a projection of the stream and the embedding's output, side by side
+                    x = cpu_ops.linear(np.concatenate([x, first], axis=-1), self.w[re.tensor_name(re.params.get("matrix", "in"))])
+                elif call.opens_pass > 0:
                     x = cpu_ops.add(x, first)
                 x = cpu_ops.add(x, np.broadcast_to(offsets[call.opens_pass], x.shape))
             owner = self.cache[call.cache_of] if call.cache_of is not None else None
             m = 0
             layer = self.spec.layers[call.layer]
-            parallel = layer.block == "parallel_residual"          # every sub-layer reads the stream as the layer found it
-            x_in = x
+            parallel = layer.block in ("parallel_residual", "shared_norm_parallel")      # every sub-layer reads the stream as the layer found it
+            x_in, h_in = x, None
             for sub in layer.sublayers:
                 src = x_in if parallel else x
                 h = self._norm(sub.norm, src) if sub.norm is not None else src
+                if layer.block == "shared_norm_parallel":          # the first sub-layer's norm serves all of them
+                    h = h_in = h if h_in is None else h_in
                 y = self._part(sub, h, positions, self.cache[c], m, owner)
                 if sub.category == "mixer":
                     m += 1
