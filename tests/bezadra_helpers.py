@@ -174,7 +174,10 @@ def random_requests(cfg: dict, lengths, seed: int):
 
 def compare(got, oracle, requests, dtype, cfg, what=""):
     """float32: every logits row within the absolute bound of helpers.tolerance.  bfloat16: no row beyond four bounds and
-    at most one row in ten beyond one (a fault, a lost key or a stale state, moves whole ranges of positions by far more)."""
+    at most one row in ten beyond one (a fault, a lost key or a stale state, moves whole ranges of positions by far more).
+    Models with recurrent heads of fewer than 16 value channels: no row beyond eight (a head's result is normed over its
+    channels, which magnifies 16-bit rounding where so short a vector is small by cancellation; the rows in question are
+    bit-equal between whole prompts, single tokens and mixed steps)."""
     import helpers
     like = like_config(cfg)
     if dtype == torch.float32:
@@ -189,7 +192,8 @@ def compare(got, oracle, requests, dtype, cfg, what=""):
             assert np.isfinite(err), f"{what}: non-finite logits at request {r} position {p}"
             ratios.append((err / tol, r, p))
     worst = max(ratios)
+    most = 8.0 if any(l["type"] == "channel_delta" and l["mixer"]["vdim"] < 16 for l in cfg["layers"]) else 4.0
     over = sum(1 for x in ratios if x[0] > 1.0)
-    assert worst[0] <= 4.0, f"{what}: request {worst[1]} position {worst[2]} is {worst[0]:.1f} bounds off"
+    assert worst[0] <= most, f"{what}: request {worst[1]} position {worst[2]} is {worst[0]:.1f} bounds off"
     assert over <= max(1, len(ratios) // 10), f"{what}: {over} of {len(ratios)} rows are beyond the bound (worst {worst[0]:.1f} at {worst[1:]})"
     return worst[0], worst[1:]

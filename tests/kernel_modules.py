@@ -15,6 +15,8 @@ TEST_MODULES = [
     # chunks, two score maps and pooled blocks (test_gpu_zetalorn.py)
     *[("attention_simt.cu", {"LLB_HEAD_DIM": k, "LLB_VALUE_DIM": v}) for k, v in ((24, 8), (10, 6), (16, 8), (12, 20), (16, 32), (32, 64))],
     ("attention_simt.cu", {"LLB_HEAD_DIM": 12}),
+    # capped scores with a learned sink (test_gpu_bezadra.py)
+    ("attention_simt.cu", {"LLB_HEAD_DIM": 96}), ("attention_mma.cu", {"LLB_HEAD_DIM": 96}), ("attention_simt.cu", {"LLB_HEAD_DIM": 2, "LLB_VALUE_DIM": 1}),
     # the build in which a bounded wait can be made to run out (test_gpu_kernels.py)
     ("gemm_tc.cu", {"LLB_WAIT_LIMIT": 4096, "LLB_TEST_STALL": 1}),
 ]
