@@ -50,7 +50,9 @@ __device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 constexpr int PREP_WARPS = 4;
-constexpr int PREP_TOKENS = 8;          // consecutive tokens of a sequence that a warp takes
+constexpr int PREP_TOKENS = 8;          // consecutive tokens of a sequence that a warp takes, or as many as the convolution
+                                        // reaches back: only a sequence's first run reads the carried inputs
+__host__ __device__ constexpr int prep_run(int taps) { return taps - 1 > PREP_TOKENS ? taps - 1 : PREP_TOKENS; }
 
 // N float32 values from / to an address aligned to N * 4 bytes.
 template <int N> __device__ __forceinline__ void load_vec(float (&v)[N], const float* src) {
@@ -64,7 +66,7 @@ template <int N> __device__ __forceinline__ void store_vec(float* dst, const flo
     else { for (int e = 0; e < N; ++e) dst[e] = v[e]; }
 }
 
-// A warp per run of 8 tokens and unit: a q, k or v head (convolution, silu, unit vector), or a head's decays and step sizes.
+// A warp per run of tokens and unit: a q, k or v head (convolution, silu, unit vector), or a head's decays and step sizes.
 // PER channels a lane: neighbours in one access (VEC: heads of 32 PER channels, aligned rows) or 32 apart.  TAPS > 0: that
 // many taps, the inputs of the run in registers; 0: any number, every input read where it is needed.  FAST: silu by the
 // special-function unit.  The warp of a sequence's first run is the only one that reads the carried inputs, and it leaves the
@@ -79,7 +81,7 @@ __device__ __forceinline__ void prep_head(const DeltaPrepParams& p, int unit, in
     float* st = p.conv_state + (size_t)p.seq_slot[b] * back * C + c0;      // [back][C]
     const float* x = p.proj + (size_t)tok0 * p.ld + c0;                    // input of the sequence's token r: x + r * ld
     float* out = p.out + (size_t)tok0 * C + c0;
-    const int hi = min(n, at0 + PREP_TOKENS);
+    const int hi = min(n, at0 + prep_run(taps));
     auto have = [&](int e) { return VEC || lane + e * 32 < d; };
     auto load = [&](float (&v)[PER], const float* src) {
         if constexpr (VEC) load_vec<PER>(v, src);
@@ -181,26 +183,30 @@ __device__ __forceinline__ void prep_head(const DeltaPrepParams& p, int unit, in
 template <int TAPS, bool FAST>
 __global__ void __launch_bounds__(PREP_WARPS * 32, 6) delta_prep_kernel(DeltaPrepParams p) {
     const int lane = threadIdx.x & 31, unit = blockIdx.y, b = blockIdx.z;
-    const int at0 = (blockIdx.x * PREP_WARPS + (threadIdx.x >> 5)) * PREP_TOKENS;
+    const int run = TAPS > 0 ? prep_run(TAPS) : prep_run(p.taps);
+    const int at0 = (blockIdx.x * PREP_WARPS + (threadIdx.x >> 5)) * run;
     const int tok0 = p.seq_start[b], n = p.seq_start[b + 1] - tok0;
     llb_grid_dependency_sync();
     if (at0 >= n) return;
     if (unit >= 2 * p.G + p.H) {                           // a head's decays and its step sizes
-        const int h = unit - 2 * p.G - p.H, C = 2 * p.G * p.dk + p.H * p.dv, m = min(PREP_TOKENS, n - at0);
+        const int h = unit - 2 * p.G - p.H, C = 2 * p.G * p.dk + p.H * p.dv;
         const float rate = expf(p.a_log[h]);
-        float* z = p.z + ((size_t)(tok0 + at0) * p.H + h) * p.dk;
         const size_t step = (size_t)p.H * p.dk;
-        if (lane < m) {
-            const size_t t = (size_t)(tok0 + at0 + lane);
-            p.beta[t * p.H + h] = 1.0f / (1.0f + expf(-p.proj[t * p.ld + C + h]));
-        }
-        for (int i = lane; i < p.dk; i += 32) {
-            float v[PREP_TOKENS];
+        for (int t0 = at0; t0 < min(n, at0 + run); t0 += PREP_TOKENS) {
+            const int m = min(min(n, at0 + run) - t0, PREP_TOKENS);
+            float* z = p.z + ((size_t)(tok0 + t0) * p.H + h) * p.dk;
+            if (lane < m) {
+                const size_t t = (size_t)(tok0 + t0 + lane);
+                p.beta[t * p.H + h] = 1.0f / (1.0f + expf(-p.proj[t * p.ld + C + h]));
+            }
+            for (int i = lane; i < p.dk; i += 32) {
+                float v[PREP_TOKENS];
 #pragma unroll
-            for (int u = 0; u < PREP_TOKENS; ++u) v[u] = u < m ? z[u * step + i] : 0.f;
+                for (int u = 0; u < PREP_TOKENS; ++u) v[u] = u < m ? z[u * step + i] : 0.f;
 #pragma unroll
-            for (int u = 0; u < PREP_TOKENS; ++u)
-                if (u < m) z[u * step + i] = expf(-rate * softplus(v[u]));
+                for (int u = 0; u < PREP_TOKENS; ++u)
+                    if (u < m) z[u * step + i] = expf(-rate * softplus(v[u]));
+            }
         }
         return;
     }
@@ -848,7 +854,7 @@ bool sizes_ok(int G, int H, int dk, int dv, int B) {
 LLB_API int llb_delta_prep(DeltaPrepParams p, int B, int max_new, cudaStream_t stream) {
     if (B == 0 || max_new == 0) return 0;
     if (!sizes_ok(p.G, p.H, p.dk, p.dv, B) || p.dv > 256 || p.taps < 1 || 2 * p.G + 2 * p.H > 65535) return (int)cudaErrorInvalidValue;
-    const int run = PREP_WARPS * PREP_TOKENS, C = 2 * p.G * p.dk + p.H * p.dv;
+    const int run = PREP_WARPS * prep_run(p.taps), C = 2 * p.G * p.dk + p.H * p.dv;
     p.vec = p.ld % 4 == 0 && C % 4 == 0 && p.dk % 4 == 0 && p.dv % 4 == 0 &&
             !(((uintptr_t)p.proj | (uintptr_t)p.conv_w | (uintptr_t)p.conv_state | (uintptr_t)p.out) & 15);
     const dim3 grid((max_new + run - 1) / run, 2 * p.G + 2 * p.H, B), block(PREP_WARPS * 32);

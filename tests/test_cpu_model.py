@@ -40,8 +40,8 @@ def test_parts_it_does_not_know_are_refused():
     from llaisys_b200.config import config_from_dict
     import dataclasses
     spec = config_from_dict(CONFIGS["A"]).to_spec()
-    odd = dataclasses.replace(spec, final_norm=dataclasses.replace(spec.final_norm, kind="layer_norm"))
-    with pytest.raises(NotImplementedError, match="layer_norm"):
+    odd = dataclasses.replace(spec, final_norm=dataclasses.replace(spec.final_norm, kind="batch_norm"))
+    with pytest.raises(NotImplementedError, match="batch_norm"):
         CpuModel(odd, {})
 
 

@@ -132,7 +132,7 @@ def _recurrent_inputs(case, b, G, H, dk, dv):
 
 
 SHAPES = [(2, 4, 16, 24, 4), (1, 3, 6, 9, 3), (2, 2, 33, 35, 1), (1, 1, 17, 7, 6), (2, 2, 64, 64, 4), (1, 2, 128, 128, 4), (1, 1, 130, 250, 4),
-          (1, 1, 256, 16, 2), (3, 3, 64, 128, 4), (1, 1, 1, 1, 4), (2, 6, 96, 40, 5)]
+          (1, 1, 256, 16, 2), (3, 3, 64, 128, 4), (1, 1, 1, 1, 4), (2, 6, 96, 40, 5), (1, 2, 16, 20, 13)]
 
 
 @pytest.mark.parametrize("shape", SHAPES, ids=[str(s) for s in SHAPES])
@@ -332,6 +332,7 @@ LAYERS = {
     "delta": bh.delta(4, 2, 16, 12, 4, bh.dense(24, 0.9)),
     "delta with one tap": bh.delta(2, 2, 8, 20, 1),
     "delta with seven taps": bh.delta(3, 1, 10, 6, 7),
+    "delta with twenty taps": bh.delta(2, 1, 64, 64, 20),
 }
 
 
