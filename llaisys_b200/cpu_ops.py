@@ -294,6 +294,25 @@ def route_grouped(logits: np.ndarray, top: int, groups=None, renorm: bool = Fals
     return idx, w * np.float32(scale)
 
 
+def route_softmax(logits: np.ndarray, bias, top: int, groups=None, scale: float = 1.0):
+    """(experts [T, top], weights [T, top]): gates softmax(z) over all logits; with groups = (count, keep) only experts of the `keep`
+    equal groups of neighbours with the largest single gate + bias can be chosen (first maximum first); the `top` largest gate +
+    bias among them; weights gate * scale (not in xsmccc/llaisys)."""
+    z = logits.astype(np.float32)
+    gate = np.exp(z - z.max(axis=-1, keepdims=True))
+    gate /= gate.sum(axis=-1, keepdims=True)
+    choice = gate if bias is None else gate + bias.astype(np.float32)
+    T, E = gate.shape
+    if groups and groups[0] > 1:
+        count, keep = groups
+        kept = np.argsort(-choice.reshape(T, count, E // count).max(axis=-1), axis=-1, kind="stable")[:, :keep]
+        allowed = np.zeros((T, count), dtype=bool)
+        np.put_along_axis(allowed, kept, True, axis=1)
+        choice = np.where(np.repeat(allowed, E // count, axis=1), choice, -np.inf)
+    idx = np.argsort(-choice, axis=-1, kind="stable")[:, :top]
+    return idx, np.take_along_axis(gate, idx, axis=-1) * np.float32(scale)
+
+
 def swish_clamped(gate: np.ndarray, up: np.ndarray, limit: float, alpha: float) -> np.ndarray:
     """g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(alpha g) (u + 1) (not in xsmccc/llaisys)."""
     g = np.minimum(gate.astype(np.float32), np.float32(limit))
@@ -346,3 +365,14 @@ def delta_recurrence(q: np.ndarray, k: np.ndarray, v: np.ndarray, g: np.ndarray,
         state += k[t][:, :, None] * u[:, None, :]
         out[t] = np.einsum("hkv,hk->hv", state, q[t])
     return out
+
+
+def state_space_recurrence(x: np.ndarray, B: np.ndarray, C: np.ndarray, step: np.ndarray, rate: np.ndarray, skip: np.ndarray, state: np.ndarray):
+    """x [T, H, P], B and C [T, H, N], step [T, H], rate and skip [H]; state [H, N, P] is updated in place:
+    S <- exp(rate step) S + step B x^T, y = S^T C + skip x; returns y [T, H, P] (not in xsmccc/llaisys)."""
+    y = np.empty_like(x)
+    for t in range(x.shape[0]):
+        state *= np.exp(rate * step[t])[:, None, None]
+        state += (step[t][:, None] * B[t])[:, :, None] * x[t][:, None, :]
+        y[t] = np.einsum("hnp,hn->hp", state, C[t]) + skip[:, None] * x[t]
+    return y

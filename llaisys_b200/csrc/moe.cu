@@ -4,14 +4,19 @@
 //   select   from the router's logits z = Wr h (float32): g = 1 / (1 + e^-z); the `top` experts with the largest
 //            g + bias are chosen (ties go to the lower index); a chosen expert's weight is g * route_scale, not
 //            renormalised.  Mode 1: the largest logits z + bias are chosen and the weights are the softmax over the
-//            chosen logits only, times route_scale.
+//            chosen logits only, times route_scale.  Mode 2: g is the softmax over all logits.  The last `identity` logits
+//            belong to identity experts, whose output is their input: they are chosen like the others, have no part in the
+//            plan, and identity_wgt[t] is the sum of their weights.
 //   plan     pair i = (token i / top, choice i % top).  Pairs are grouped by expert: slot_of[pair] is a pair's place
 //            in that order, pair_of[slot] its inverse, and every expert's run of slots is cut into tiles of
 //            `tile_rows` rows (tile -> expert, first slot, rows), so that the products run over a grid whose size
-//            depends on the step's shape alone and never on the routing (a captured step stays valid).
+//            depends on the step's shape alone and never on the routing (a captured step stays valid).  Pairs of experts
+//            outside 0 .. E - 1 (identity experts) take the slots behind all others and no tile; n_tiles[1] counts the
+//            slots before them.
 //   product  out[slot, :] = act(A[row(slot), :] W[expert(slot)]^T) on the CUDA cores, float32 accumulation (the true
 //            32-bit path, and the bfloat16 path wherever the tensor-core kernel below does not apply).
 //   combine  stream[t, :] += sum_k weight[t, k] * y[slot_of[t top + k], :], k in order: deterministic.
+//   identity out[t, :] = (or +=) identity_wgt[t] * x[t, :].
 #include "common.cuh"
 
 constexpr int MOE_TILE = 64;
@@ -22,7 +27,8 @@ constexpr int MOE_TILE = 64;
 // arg-max (ties to the lower index), weights g * route_scale.
 __global__ void __launch_bounds__(128)
 moe_select_kernel(const float* __restrict__ z, int ldz, const float* __restrict__ bias, int T, int E, int top, float route_scale,
-                  int* __restrict__ idx, float* __restrict__ wgt, int mode, int n_groups, int keep_groups, int renorm) {
+                  int* __restrict__ idx, float* __restrict__ wgt, int mode, int n_groups, int keep_groups, int group_max, int renorm,
+                  int identity, float* __restrict__ identity_wgt) {
     extern __shared__ float sm[];                 // per warp: gate[E], choice[E]
     __shared__ float group_score[4][64];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -31,16 +37,25 @@ moe_select_kernel(const float* __restrict__ z, int ldz, const float* __restrict_
     float* choice = gate + E;
     llb_grid_dependency_sync();
     if (t >= T) return;
+    float top_z = 0.f, inv_sum = 1.f;
+    if (mode == 2) {
+        top_z = -INFINITY;
+        for (int e = lane; e < E; e += 32) top_z = fmaxf(top_z, z[(size_t)t * ldz + e]);
+        top_z = warp_max(top_z);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) sum += expf(z[(size_t)t * ldz + e] - top_z);
+        inv_sum = 1.0f / warp_sum(sum);
+    }
     for (int e = lane; e < E; e += 32) {
         const float zl = z[(size_t)t * ldz + e];
-        const float g = mode == 1 ? zl : 1.0f / (1.0f + expf(-zl));
+        const float g = mode == 1 ? zl : mode == 2 ? expf(zl - top_z) * inv_sum : 1.0f / (1.0f + expf(-zl));
         gate[e] = g;
         choice[e] = g + (bias ? bias[e] : 0.f);
     }
     __syncwarp();
     if (n_groups > 1) {
         // the experts form n_groups equal groups of neighbours; a group's score is the sum of its two largest choice
-        // scores; only experts of the keep_groups best groups (first maximum first) stay in the choice
+        // scores (group_max: its largest one); only experts of the keep_groups best groups (first maximum first) stay in the choice
         const int per = E / n_groups;
         float* gs = group_score[warp];
         for (int g = lane; g < n_groups; g += 32) {
@@ -50,7 +65,7 @@ moe_select_kernel(const float* __restrict__ z, int ldz, const float* __restrict_
                 if (c > b0) { b1 = b0; b0 = c; }
                 else if (c > b1) b1 = c;
             }
-            gs[g] = per > 1 ? b0 + b1 : b0;
+            gs[g] = per > 1 && !group_max ? b0 + b1 : b0;
         }
         __syncwarp();
         if (lane == 0) {
@@ -105,6 +120,12 @@ moe_select_kernel(const float* __restrict__ z, int ldz, const float* __restrict_
         const float inv = route_scale / sum;
         for (int k = 0; k < top; ++k) w[k] *= inv;
     }
+    if (identity_wgt && lane == 0) {
+        float sum = 0.f;
+        for (int k = 0; k < top; ++k)
+            if (idx[(size_t)t * top + k] >= E - identity) sum += wgt[(size_t)t * top + k];
+        identity_wgt[t] = sum;
+    }
     if (mode != 1 && renorm && lane == 0) {
         // the chosen gates divided by their sum (the factor route_scale is in them already)
         float* w = wgt + (size_t)t * top;
@@ -116,19 +137,20 @@ moe_select_kernel(const float* __restrict__ z, int ldz, const float* __restrict_
 }
 
 LLB_API int llb_moe_select(const float* z, int ldz, const float* bias, int T, int E, int top, float route_scale, int* idx,
-                           float* wgt, int mode, int n_groups, int keep_groups, int renorm, cudaStream_t stream) {
+                           float* wgt, int mode, int n_groups, int keep_groups, int group_max, int renorm, int identity, float* identity_wgt,
+                           cudaStream_t stream) {
     if (T == 0) return 0;
-    if (top < 1 || top > E) return (int)cudaErrorInvalidValue;
+    if (top < 1 || top > E || identity < 0 || identity > E || (identity_wgt && (mode == 1 || renorm))) return (int)cudaErrorInvalidValue;
     if (n_groups > 1 && (n_groups > 64 || E % n_groups || keep_groups < 1 || keep_groups > n_groups)) return (int)cudaErrorInvalidValue;
     const size_t smem = (size_t)4 * 2 * E * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     llb_launch(moe_select_kernel, dim3((T + 3) / 4), dim3(128), smem, stream, z, ldz, bias, T, E, top, route_scale, idx, wgt, mode,
-               n_groups, keep_groups, renorm);
+               n_groups, keep_groups, group_max, renorm, identity, identity_wgt);
     return llb_status();
 }
 
 // ------------------------------------------------------------------ plan
-// One block.  tiles: int32 [3, max_tiles] (expert, first slot, rows) and n_tiles [1]; max_tiles >= N / tile_rows + min(E, N).
+// One block.  tiles: int32 [3, max_tiles] (expert, first slot, rows) and n_tiles [2] (tiles, slots that are in one); max_tiles >= N / tile_rows + min(E, N).
 __global__ void __launch_bounds__(1024)
 moe_plan_kernel(const int* __restrict__ idx, int N, int E, int tile_rows, int* __restrict__ slot_of, int* __restrict__ pair_of,
                 int* __restrict__ tiles, int max_tiles, int* __restrict__ n_tiles) {
@@ -137,6 +159,7 @@ moe_plan_kernel(const int* __restrict__ idx, int N, int E, int tile_rows, int* _
     int* first = count + E;
     int* cursor = first + E;
     int* tile0 = cursor + E;
+    __shared__ int outside, inside;
     const int tid = threadIdx.x;
     for (int e = tid; e < E; e += blockDim.x) count[e] = cursor[e] = 0;
     llb_grid_dependency_sync();
@@ -160,7 +183,9 @@ moe_plan_kernel(const int* __restrict__ idx, int N, int E, int tile_rows, int* _
             tl += (count[e] + tile_rows - 1) / tile_rows;
         }
         tile0[E] = tl;
-        *n_tiles = min(tl, max_tiles);
+        n_tiles[0] = min(tl, max_tiles);
+        n_tiles[1] = inside = f;
+        outside = 0;
     }
     __syncthreads();
     for (int e = tid; e < E; e += blockDim.x) {
@@ -177,8 +202,8 @@ moe_plan_kernel(const int* __restrict__ idx, int N, int E, int tile_rows, int* _
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
             const int e = e4[u], i = i0 + u * blockDim.x;
-            if (e < 0 || e >= E) continue;
-            const int s = first[e] + atomicAdd(&cursor[e], 1);
+            if (i >= N) continue;
+            const int s = e >= 0 && e < E ? first[e] + atomicAdd(&cursor[e], 1) : inside + atomicAdd(&outside, 1);
             slot_of[i] = s;
             pair_of[s] = i;
         }
@@ -298,9 +323,11 @@ LLB_API int llb_moe_gemm(const void* A, int a_dtype, int lda, const int* pair_of
 // box).  16-byte pieces where the rows allow it.
 template <typename T>
 __global__ void __launch_bounds__(256)
-moe_gather_rows_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ pair_of, int top, T* __restrict__ out, int H) {
+moe_gather_rows_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ pair_of, int top, const int* __restrict__ n_tiles,
+                       T* __restrict__ out, int H) {
     llb_grid_dependency_sync();
     const int slot = blockIdx.x;
+    if (slot >= n_tiles[1]) return;
     const T* src = x + (size_t)(pair_of[slot] / top) * ldx;
     T* dst = out + (size_t)slot * H;
     constexpr int V = 16 / sizeof(T);
@@ -312,11 +339,12 @@ moe_gather_rows_kernel(const T* __restrict__ x, int ldx, const int* __restrict__
     }
 }
 
-LLB_API int llb_moe_gather_rows(const void* x, int dtype, int ldx, const int* pair_of, int top, void* out, int n_slots, int H,
+LLB_API int llb_moe_gather_rows(const void* x, int dtype, int ldx, const int* pair_of, int top, const int* n_tiles, void* out, int n_slots, int H,
                                 cudaStream_t stream) {
     if (n_slots == 0) return 0;
     LLB_DISPATCH_DTYPE(dtype, T,
-        llb_launch(moe_gather_rows_kernel<T>, dim3(n_slots), dim3(256), 0, stream, (const T*)x, ldx, pair_of, top, (T*)out, H));
+        llb_launch(moe_gather_rows_kernel<T>, dim3(n_slots), dim3(256), 0, stream, (const T*)x, ldx, pair_of, top, n_tiles,
+                   (T*)out, H));
     return llb_status();
 }
 
@@ -324,21 +352,59 @@ LLB_API int llb_moe_gather_rows(const void* x, int dtype, int ldx, const int* pa
 template <typename TY>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(float* __restrict__ stream, const TY* __restrict__ y, int ldy, const int* __restrict__ slot_of,
-                   const float* __restrict__ wgt, int top, int H) {
+                   const float* __restrict__ wgt, int top, const int* __restrict__ n_tiles, int H) {
     llb_grid_dependency_sync();
-    const int t = blockIdx.x;
+    const int t = blockIdx.x, inside = n_tiles[1];
     for (int j = threadIdx.x; j < H; j += blockDim.x) {
         float acc = 0.f;
-        for (int k = 0; k < top; ++k)
-            acc = fmaf(wgt[(size_t)t * top + k], to_f32(y[(size_t)slot_of[(size_t)t * top + k] * ldy + j]), acc);
+        for (int k = 0; k < top; ++k) {
+            const int slot = slot_of[(size_t)t * top + k];
+            if (slot < inside) acc = fmaf(wgt[(size_t)t * top + k], to_f32(y[(size_t)slot * ldy + j]), acc);
+        }
         stream[(size_t)t * H + j] += acc;
     }
 }
 
 LLB_API int llb_moe_combine(float* stream, const void* y, int y_dtype, int ldy, const int* slot_of, const float* wgt, int T,
-                            int top, int H, cudaStream_t stream_) {
+                            int top, const int* n_tiles, int H, cudaStream_t stream_) {
     if (T == 0) return 0;
     LLB_DISPATCH_DTYPE(y_dtype, TY,
-        llb_launch(moe_combine_kernel<TY>, dim3(T), dim3(256), 0, stream_, stream, (const TY*)y, ldy, slot_of, wgt, top, H));
+        llb_launch(moe_combine_kernel<TY>, dim3(T), dim3(256), 0, stream_, stream, (const TY*)y, ldy, slot_of, wgt, top,
+                   n_tiles, H));
+    return llb_status();
+}
+
+// ------------------------------------------------------------------ identity experts
+template <typename T, bool ADD>
+__global__ void __launch_bounds__(256) moe_identity_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ w, float* __restrict__ out,
+                                                           int ldo, int H) {
+    llb_grid_dependency_sync();
+    const int t = blockIdx.x;
+    const float wt = w[t];
+    const T* src = x + (size_t)t * ldx;
+    float* dst = out + (size_t)t * ldo;
+    if (ADD && wt == 0.f) return;
+    if (H % 4 == 0 && ldx % 4 == 0 && ldo % 4 == 0 && !(((uintptr_t)x | (uintptr_t)out) & 15)) {
+        struct alignas(4 * sizeof(T)) Four { T v[4]; };
+        for (int j = threadIdx.x * 4; j < H; j += 1024) {
+            const Four q = *reinterpret_cast<const Four*>(src + j);
+            float4 y = ADD ? *reinterpret_cast<const float4*>(dst + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            y.x = fmaf(wt, to_f32(q.v[0]), y.x);
+            y.y = fmaf(wt, to_f32(q.v[1]), y.y);
+            y.z = fmaf(wt, to_f32(q.v[2]), y.z);
+            y.w = fmaf(wt, to_f32(q.v[3]), y.w);
+            *reinterpret_cast<float4*>(dst + j) = y;
+        }
+        return;
+    }
+    for (int j = threadIdx.x; j < H; j += 256) dst[j] = fmaf(wt, to_f32(src[j]), ADD ? dst[j] : 0.f);
+}
+
+LLB_API int llb_moe_identity(const void* x, int dtype, int ldx, const float* w, float* out, int ldo, int T, int H, int add, cudaStream_t stream) {
+    if (T == 0) return 0;
+    LLB_DISPATCH_DTYPE(dtype, TT, {
+        if (add) llb_launch(moe_identity_kernel<TT, true>, dim3(T), dim3(256), 0, stream, (const TT*)x, ldx, w, out, ldo, H);
+        else llb_launch(moe_identity_kernel<TT, false>, dim3(T), dim3(256), 0, stream, (const TT*)x, ldx, w, out, ldo, H);
+    });
     return llb_status();
 }

@@ -5,6 +5,7 @@
 //   branch_mean   out[r] = mult * sum_b x_b[r] / sqrt(mean(x_b[r]^2) + eps) * w_b: several mixers' results, each normed
 //                 over the row with a weight of its own, averaged
 //   scale_rows    x *= c
+//   softcap_rows  x <- c tanh(x / c)
 //   layer_norm    out[r] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * weight, v = x[rows ? rows[r] : r]
 //   copy_rows     rows of the stream, converted, into a matrix of another row stride
 //
@@ -311,5 +312,17 @@ __global__ void scale_rows_kernel(float* __restrict__ x, size_t n, float c) {
 LLB_API int llb_scale_rows(float* x, long long n, float c, cudaStream_t stream) {
     if (n == 0) return 0;
     llb_launch(scale_rows_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, x, (size_t)n, c);
+    return llb_status();
+}
+
+__global__ void softcap_rows_kernel(float* __restrict__ x, size_t n, float c) {
+    llb_grid_dependency_sync();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) x[i] = c * tanhf(x[i] / c);
+}
+
+LLB_API int llb_softcap_rows(float* x, long long n, float c, cudaStream_t stream) {
+    if (n == 0) return 0;
+    llb_launch(softcap_rows_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, x, (size_t)n, c);
     return llb_status();
 }

@@ -161,6 +161,15 @@ def scale_(x: torch.Tensor, c: float) -> torch.Tensor:
     return x
 
 
+def softcap_(x: torch.Tensor, c: float) -> torch.Tensor:
+    """x <- c tanh(x / c) in place (float32, contiguous)."""
+    _need_cuda(x)
+    assert x.dtype == torch.float32 and x.is_contiguous() and c > 0
+    f = _fn(load_module("streamops.cu"), "llb_softcap_rows", [c_void_p, c_longlong, c_float, c_void_p])
+    _check(f(_ptr(x), x.numel(), c, _stream()), "cap")
+    return x
+
+
 def layer_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
     """(x - mean) / sqrt(mean((x - mean)^2) + eps) * weight over the rows of the float32 stream x [T, H], in out_dtype; with
     rows (int32) only those rows, [len(rows), H]."""

@@ -1,4 +1,5 @@
-"""Python faces of the kernels of the recurrent and the latent mixers (csrc/gla.cu, csrc/delta.cu, csrc/headout.cu, csrc/latent.cu, and the CUDA-core
+"""Python faces of the kernels of the recurrent and the latent mixers (csrc/gla.cu, csrc/delta.cu, csrc/shortconv.cu, csrc/ssd.cu, csrc/headout.cu,
+csrc/latent.cu, and the CUDA-core
 attention kernel of csrc/attention_simt.cu run over a cache of latent rows)."""
 from __future__ import annotations
 
@@ -186,6 +187,130 @@ def delta_scan(qkv: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: to
     f = _fn(lib, "llb_delta_chunked", [_DeltaChunkParams, c_int, c_int, c_int, c_void_p])
     _check(f(p, n_seqs, max_new, _sm_count(qkv.device), _stream()), "delta rule (recurrence in chunks)", 2)
     del rec
+    return out
+
+
+class _ShortConvParams(ctypes.Structure):
+    _fields_ = [("x", c_void_p), ("ld", c_int), ("w", c_void_p), ("bias", c_void_p), ("state", c_void_p), ("seq_start", c_void_p),
+                ("seq_slot", c_void_p), ("C", c_int), ("taps", c_int)]
+
+
+class _ConvHeadsParams(ctypes.Structure):
+    _fields_ = [("conv", _ShortConvParams), ("out", c_void_p), ("ldo", c_int), ("n_q", c_int), ("n_k", c_int), ("d", c_int), ("rot", c_int),
+                ("v_mult", c_float), ("cos_t", c_void_p), ("sin_t", c_void_p), ("table_rows", c_int), ("tok_pos", c_void_p),
+                ("append", c_int), ("seq_len_before", c_void_p), ("kpool", c_void_p), ("vpool", c_void_p), ("page_table", c_void_p),
+                ("table_stride", c_int), ("ring", c_int), ("pinned", c_int), ("err", c_void_p)]
+
+
+def _conv_params(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor], ctx) -> _ShortConvParams:
+    _need_cuda(x, w, bias, state)
+    taps, C = w.shape
+    assert x.stride(1) == 1 and x.shape[1] == C and w.dtype == torch.float32 and w.is_contiguous()
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == C and bias.is_contiguous())
+    assert taps == 1 or (state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == (taps - 1) * C)
+    p = _ShortConvParams()
+    p.x, p.ld, p.w, p.bias, p.state = x.data_ptr(), x.stride(0), w.data_ptr(), _ptr(bias), _ptr(state) if taps > 1 else None
+    p.seq_start, p.seq_slot, p.C, p.taps = ctx.seq_start.data_ptr(), ctx.seq_slot.data_ptr(), C, taps
+    return p
+
+
+def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor], ctx, act: Optional[str] = None,
+               out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """The causal convolution of every channel of x [T, C] (row stride free) over its sequence's tokens, plus bias (float32 [C] or
+    None), then act (None or "silu"): [T, C] in out_dtype.  w float32 [taps, C], the last row for the current token; state (float32
+    [slots, (taps - 1) C], oldest input first; None with one tap) holds each sequence's last inputs and is brought up to date."""
+    p = _conv_params(x, w, bias, state, ctx)
+    out = torch.empty((x.shape[0], p.C), dtype=out_dtype or x.dtype, device=x.device)
+    f = _fn(load_module("shortconv.cu"), "llb_short_conv", [_ShortConvParams, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(p, _dt(x), _ptr(out), _dt(out), out.stride(0), {None: 0, "silu": 1}[act], ctx.n_seqs, ctx.max_new, _stream()), "short convolution")
+    return out
+
+
+def conv_heads(x: torch.Tensor, n_q: int, n_k: int, d: int, w: torch.Tensor, state: Optional[torch.Tensor], ctx, tables=None,
+               v_mult: float = 1.0, append: Optional[dict] = None) -> torch.Tensor:
+    """From the projections x [T, (n_q + n_k) d] of query and key heads, each channel through a causal convolution (w, state as for
+    short_conv): packed [T, (n_q + 2 n_k) d] with the queries and keys, their first `dims` dimensions rotated in pairs
+    (i, i + dims / 2) by tables = (cos, sin, dims), and the values: the convolved keys before the rotation, times v_mult.  append =
+    dict(seq_len_before, kpool, vpool, page_table, ring, pinned): the keys and values also go into the paged cache."""
+    T = x.shape[0]
+    p = _ConvHeadsParams()
+    p.conv = _conv_params(x, w, None, state, ctx)
+    out = torch.empty((T, (n_q + 2 * n_k) * d), dtype=x.dtype, device=x.device)
+    p.out, p.ldo, p.n_q, p.n_k, p.d, p.v_mult = out.data_ptr(), out.stride(0), n_q, n_k, d, v_mult
+    if tables is not None:
+        cos, sin, dims = tables
+        assert cos.dtype == sin.dtype == torch.float32 and cos.shape[1] == dims // 2 and cos.is_contiguous() and sin.is_contiguous()
+        p.rot, p.cos_t, p.sin_t, p.table_rows = dims, cos.data_ptr(), sin.data_ptr(), cos.shape[0]
+    p.tok_pos, p.err = ctx.tok_pos.data_ptr(), ctx.err.data_ptr()
+    if append is not None:
+        a = append
+        assert a["kpool"].dtype == a["vpool"].dtype == x.dtype
+        p.append, p.seq_len_before, p.kpool, p.vpool = 1, a["seq_len_before"].data_ptr(), a["kpool"].data_ptr(), a["vpool"].data_ptr()
+        p.page_table, p.table_stride, p.ring, p.pinned = a["page_table"].data_ptr(), a["page_table"].shape[1], a["ring"], a.get("pinned", 0)
+    f = _fn(load_module("shortconv.cu"), "llb_conv_heads", [_ConvHeadsParams, c_int, c_int, c_int, c_void_p])
+    _check(f(p, _dt(x), ctx.n_seqs, ctx.max_new, _stream()), "short convolution, rotation and cache append of heads")
+    return out
+
+
+class _SsdParams(ctypes.Structure):
+    _fields_ = [("xbc", c_void_p), ("ld", c_int), ("dt", c_void_p), ("dt_ld", c_int), ("dt_bias", c_void_p), ("a_log", c_void_p),
+                ("skip", c_void_p), ("state", c_void_p), ("seq_start", c_void_p), ("seq_slot", c_void_p), ("out", c_void_p),
+                ("H", c_int), ("P", c_int), ("N", c_int), ("G", c_int), ("rec", c_void_p), ("decay", c_void_p)]
+
+
+SSD_MAX_STATE = 256           # rows of a head's state
+SSD_CHUNKED_FROM = 32         # steps whose longest sequence brings at least this many tokens run in chunks
+
+
+def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor,
+             seq_start: torch.Tensor, seq_slot: torch.Tensor, n_seqs: int, max_new: int, H: int, P: int, N: int, G: int,
+             chunked: bool = False) -> torch.Tensor:
+    """The state-space recurrence over the new tokens of every sequence: xbc [T, H P + 2 G N] holds x (H heads of P), B and C (G
+    groups of N); dt (float32 [T, H], row stride free) the logits of the step sizes softplus(dt + dt_bias); S <- exp(-exp(a_log)
+    step) S + step B x^T, y = S^T C + skip x; state [slots, H N P] (float32) is read at row seq_slot[b] and left holding the state
+    after the step.  Returns y [T, H P] in float32.  chunked (bfloat16 xbc): chunks of 64 tokens on the tensor cores instead of token
+    by token on the CUDA cores."""
+    _need_cuda(xbc, dt, dt_bias, a_log, skip, state)
+    T = xbc.shape[0]
+    assert xbc.stride(1) == 1 and xbc.shape[1] == H * P + 2 * G * N and dt.dtype == torch.float32 and dt.shape == (T, H) and dt.stride(1) == 1
+    for v in (dt_bias, a_log, skip):
+        assert v.dtype == torch.float32 and v.numel() == H and v.is_contiguous()
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == H * N * P
+    if N > SSD_MAX_STATE:
+        raise KernelError(f"state space: {N} state rows a head; the kernels take up to {SSD_MAX_STATE}")
+    out = torch.empty((T, H * P), dtype=torch.float32, device=xbc.device)
+    p = _SsdParams()
+    p.xbc, p.ld, p.dt, p.dt_ld = xbc.data_ptr(), xbc.stride(0), dt.data_ptr(), dt.stride(0)
+    p.dt_bias, p.a_log, p.skip, p.state = dt_bias.data_ptr(), a_log.data_ptr(), skip.data_ptr(), state.data_ptr()
+    p.seq_start, p.seq_slot, p.out, p.H, p.P, p.N, p.G = seq_start.data_ptr(), seq_slot.data_ptr(), out.data_ptr(), H, P, N, G
+    lib = load_module("ssd.cu")
+    if not chunked:
+        f = _fn(lib, "llb_ssd_scan", [_SsdParams, c_int, c_int, c_void_p])
+        _check(f(p, _dt(xbc), n_seqs, _stream()), "state space (recurrence)")
+        return out
+    assert xbc.dtype == torch.bfloat16
+    chunks = _fn(lib, "llb_ssd_chunks", [c_int, c_int])(T, n_seqs)
+    rec = torch.empty((chunks, H * N * P), dtype=torch.float32, device=xbc.device)
+    decay = torch.empty((chunks, H), dtype=torch.float32, device=xbc.device)
+    p.rec, p.decay = rec.data_ptr(), decay.data_ptr()
+    f = _fn(lib, "llb_ssd_chunked", [_SsdParams, c_int, c_int, c_void_p])
+    _check(f(p, n_seqs, max_new, _stream()), "state space (recurrence in chunks)", 3)
+    del rec, decay
+    return out
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """[T, C]: g = y * silu(z) (y float32, z a view with any row stride), each of `groups` equal parts of the row divided by its own
+    sqrt(mean(g^2) + eps), times weight (float32 [C])."""
+    _need_cuda(y, z, weight)
+    T, C = y.shape
+    assert y.dtype == torch.float32 and y.is_contiguous() and z.shape == (T, C) and z.stride(1) == 1
+    assert weight.dtype == torch.float32 and weight.numel() == C and weight.is_contiguous() and groups > 0 and C % groups == 0
+    out = torch.empty((T, C), dtype=out_dtype, device=y.device)
+    f = _fn(load_module("ssd.cu"), "llb_gated_group_norm", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                                            c_float, c_void_p])
+    _check(f(_ptr(y), _ptr(z), _dt(z), z.stride(0), _ptr(weight), _ptr(out), DT[out_dtype], T, groups, C // groups, eps, _stream()),
+           "gate and norm in parts")
     return out
 
 

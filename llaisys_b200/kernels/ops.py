@@ -533,6 +533,7 @@ class GluForm:
 
 
 SWIGLU = GluForm()
+RELU_GLU = GluForm(alpha=1e30)        # g / (1 + e^(-1e30 g)) is max(g, 0): the gate of a ReLU feed-forward
 
 
 def _gemm_tc_pair(x, weight, bias, out, dual_offset=0, glu=SWIGLU):
@@ -661,6 +662,8 @@ def linear_swiglu(x: torch.Tensor, gate_up: torch.Tensor, plan=None, form: GluFo
         return out
     if form == SWIGLU:
         return swiglu(linear(x, gate_up))
+    if form == RELU_GLU:
+        return glu(linear(x, gate_up), "relu")
     if form.plus != 1.0:
         raise KernelError(f"gated activation: no kernel of its own combines gate and up as {form}")
     return glu(linear(x, gate_up), "swish_clamped", limit=form.limit, alpha=form.alpha)
@@ -1084,12 +1087,23 @@ def moe_tile_rows() -> int:
     return _moe_tile
 
 
-MOE_GATES = {"sigmoid": 0, "softmax_chosen": 1}
+MOE_GATES = {"sigmoid": 0, "softmax_chosen": 1, "softmax": 2}
+
+
+def narrow_plan(x: torch.Tensor, weight: torch.Tensor):
+    """The plan of a float32 product of many tokens with a handful of rows: tiles of 64 tokens and the K range cut over a cluster, so
+    that it runs on more than T / 256 blocks.  None where linear() chooses by itself."""
+    T, H = x.shape
+    if T <= 256 or not _tc_ok(x, weight, None):
+        return None
+    tiles, kblocks = -(-T // 64) * -(-weight.shape[0] // 128), -(-H // 64)
+    splits = max([s for s in (1, 2, 4, 8) if s == 1 or (tiles * s <= 2 * _sm_count(x.device) and s <= kblocks // 2)])
+    return (64, splits)
 
 
 def moe_route(x: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor], top: int, route_scale: float,
               gate: str = "sigmoid", n_experts: Optional[int] = None, with_logits: bool = False, groups: Optional[tuple] = None,
-              renorm: bool = False):
+              renorm: bool = False, group_max: bool = False, identity: int = 0):
     """(int32 [T, top] experts, float32 [T, top] weights): the router's logits x router^T in float32 (a matrix product
     with float32 accumulation: on the tensor cores for bfloat16 operands, on the CUDA cores in float32).  gate "sigmoid":
     gates sigmoid(logits); the `top` largest of gate + bias are chosen (first maximum first); a weight is
@@ -1098,31 +1112,28 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor
     (other per-token logits that ride on the same product); with_logits also returns all logits [T, rows] (float32).
     groups = (count, keep): the experts form `count` equal groups of neighbours, a group's score is the sum of its two
     largest choice scores, and only experts of the `keep` best groups can be chosen.  renorm (gate "sigmoid"): the chosen
-    gates are divided by their sum (+ 1e-20) before route_scale is applied."""
+    gates are divided by their sum (+ 1e-20) before route_scale is applied.  gate "softmax": as "sigmoid", with gates that are the
+    softmax over all logits.  group_max: a group's score is its largest choice score.  identity: the last so many of the logits
+    belong to experts whose output is their input; a chosen one keeps its number in the result, and the sum of such weights is
+    returned as one more float32 [T] at the end."""
     _need_cuda(x, router, bias)
     T, H = x.shape
     rows = router.shape[0]
     E = rows if n_experts is None else int(n_experts)
     assert router.shape == (rows, H) and E <= rows and router.is_contiguous() and x.stride(1) == 1
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == E)
-    plan = None
-    if T > 256 and _tc_ok(x, router, None):
-        # many tokens against a handful of rows: tiles of 64 tokens and the K range cut over a cluster, so that the
-        # product runs on more than T / 256 blocks
-        tiles, kblocks = -(-T // 64) * -(-rows // 128), -(-H // 64)
-        splits = max([s for s in (1, 2, 4, 8) if s == 1 or (tiles * s <= 2 * _sm_count(x.device) and s <= kblocks // 2)])
-        plan = (64, splits)
-    z = linear(x, router, out_dtype=torch.float32, plan=plan)
+    z = linear(x, router, out_dtype=torch.float32, plan=narrow_plan(x, router))
     idx = torch.empty((T, top), dtype=torch.int32, device=x.device)
     wgt = torch.empty((T, top), dtype=torch.float32, device=x.device)
+    w_id = torch.empty((T,), dtype=torch.float32, device=x.device) if identity else None
     n_groups, keep_groups = (int(groups[0]), int(groups[1])) if groups else (1, 1)
     if n_groups > 1 and (E % n_groups or not (1 <= keep_groups <= n_groups) or n_groups > 64):
         raise KernelError(f"router: {E} experts in {n_groups} groups of which {keep_groups} are kept cannot be (equal groups, at most 64)")
     f = _fn(_moe_lib(), "llb_moe_select", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int,
-                                           c_int, c_int, c_int, c_void_p])
+                                           c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
     _check(f(_ptr(z), z.stride(0), _ptr(bias), T, E, top, route_scale, _ptr(idx), _ptr(wgt), MOE_GATES[gate], n_groups, keep_groups,
-             int(renorm), _stream()), "router's choice")
-    return (idx, wgt, z) if with_logits else (idx, wgt)
+             int(group_max), int(renorm), identity, _ptr(w_id), _stream()), "router's choice")
+    return (idx, wgt) + ((z,) if with_logits else ()) + ((w_id,) if identity else ())
 
 
 class MoePlan:
@@ -1138,7 +1149,7 @@ def moe_plan(idx: torch.Tensor, n_experts: int, tile_rows: Optional[int] = None)
     p = MoePlan()
     p.top, p.n_pairs, p.tile_rows = top, N, int(tile_rows or moe_tile_rows())
     p.max_tiles = N // p.tile_rows + min(n_experts, N)       # an expert that has pairs ends in one partial tile at most
-    buf = torch.empty(2 * N + 3 * p.max_tiles + 1, dtype=torch.int32, device=idx.device)
+    buf = torch.empty(2 * N + 3 * p.max_tiles + 2, dtype=torch.int32, device=idx.device)
     p.slot_of, p.pair_of = buf[:N], buf[N:2 * N]
     p.tiles, p.n_tiles = buf[2 * N:2 * N + 3 * p.max_tiles], buf[2 * N + 3 * p.max_tiles:]
     f = _fn(_moe_lib(), "llb_moe_plan", [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p])
@@ -1182,8 +1193,8 @@ def moe_gather_rows(x: torch.Tensor, plan: MoePlan) -> torch.Tensor:
     _need_cuda(x)
     assert x.stride(1) == 1
     out = torch.empty((plan.n_pairs, x.shape[1]), dtype=x.dtype, device=x.device)
-    f = _fn(_moe_lib(), "llb_moe_gather_rows", [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p])
-    _check(f(_ptr(x), _dt(x), x.stride(0), _ptr(plan.pair_of), plan.top, _ptr(out), plan.n_pairs, x.shape[1], _stream()),
+    f = _fn(_moe_lib(), "llb_moe_gather_rows", [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p])
+    _check(f(_ptr(x), _dt(x), x.stride(0), _ptr(plan.pair_of), plan.top, _ptr(plan.n_tiles), _ptr(out), plan.n_pairs, x.shape[1], _stream()),
            "experts' rows in slot order")
     return out
 
@@ -1217,9 +1228,21 @@ def moe_combine(stream: torch.Tensor, y: torch.Tensor, plan: MoePlan, wgt: torch
     _need_cuda(stream, y, wgt)
     T, H = stream.shape
     assert stream.dtype == torch.float32 and stream.is_contiguous() and y.shape[1] == H and y.stride(1) == 1
-    f = _fn(_moe_lib(), "llb_moe_combine", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
-    _check(f(_ptr(stream), _ptr(y), _dt(y), y.stride(0), _ptr(plan.slot_of), _ptr(wgt), T, plan.top, H, _stream()),
+    f = _fn(_moe_lib(), "llb_moe_combine", [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p])
+    _check(f(_ptr(stream), _ptr(y), _dt(y), y.stride(0), _ptr(plan.slot_of), _ptr(wgt), T, plan.top, _ptr(plan.n_tiles), H, _stream()),
            "experts' weighted sum")
+
+
+def moe_identity(x: torch.Tensor, w: torch.Tensor, stream: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """stream[t] += w[t] * x[t] (float32 stream [T, H]); without a stream the product is returned as a new float32 tensor."""
+    _need_cuda(x, w, stream)
+    T, H = x.shape
+    assert x.stride(1) == 1 and w.dtype == torch.float32 and w.numel() == T and w.is_contiguous()
+    out = stream if stream is not None else torch.empty((T, H), dtype=torch.float32, device=x.device)
+    assert out.dtype == torch.float32 and out.shape == (T, H) and out.stride(1) == 1
+    f = _fn(_moe_lib(), "llb_moe_identity", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(x), _dt(x), x.stride(0), _ptr(w), _ptr(out), out.stride(0), T, H, int(stream is not None), _stream()), "identity experts")
+    return out
 
 
 # ------------------------------------------------------------------ choice of the next token

@@ -21,7 +21,7 @@ from ..config.spec import ModelSpec, PartSpec
 _KNOWN = {"embedding": {"token_embedding", "scaled_pair_embedding"}, "norm": {"rms_norm", "layer_norm"},
           "mixer": {"gqa_attention", "windowed_sink_attention", "gated_linear_attention", "latent_attention", "min_gru",
                     "differential_attention", "pooled_window_attention", "lightning_attention", "parallel_mixers",
-                    "channel_delta_rule"},
+                    "channel_delta_rule", "state_space"},
           "ffn": {"swiglu_mlp", "routed_experts", "gated_mlp"},
           "block": {"pre_norm_residual", "parallel_residual", "sandwich_residual", "depth_averaged_residual", "gated_residual",
                     "shared_norm_parallel"},
@@ -116,6 +116,29 @@ class CpuModel:
         o = cpu_ops.delta_recurrence(np.repeat(q, H // G, axis=1), np.repeat(k, H // G, axis=1), v, g, cpu_ops.sigmoid(cpu_ops.linear(x, w("b"))), S)
         o = cpu_ops.rms_norm(o, w("norm"), a["eps"]).reshape(T, H * dv)
         return cpu_ops.linear(o * cpu_ops.sigmoid(cpu_ops.linear(cpu_ops.linear(x, w("g1")), w("g2"))), w("o"))
+
+    def _state_space(self, p: PartSpec, x, store: dict, key):
+        a = p.params
+        H, P, N, G, taps = a["num_heads"], a["value_dim"], a["state"], a["groups"], a["taps"]
+        n = dict({"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "A_log": "A_log", "D": "D", "norm": "norm",
+                  "o": "o"}, **(a.get("names") or {}))
+        w = lambda k: self.w[p.tensor_name(n[k])].astype(np.float32)
+        T, inner = x.shape[0], H * P
+        proj = cpu_ops.linear(x, w("in"))
+        z, raw, dt = proj[:, :inner], proj[:, inner:2 * inner + 2 * G * N], proj[:, 2 * inner + 2 * G * N:]
+        if key not in store:
+            store[key] = (np.zeros((H, N, P), dtype=np.float32), np.zeros((taps - 1, raw.shape[1]), dtype=np.float32))
+        S, last = store[key]
+        y, last[:] = cpu_ops.causal_conv(raw, w("conv"), last)
+        y = y + w("conv_bias")
+        y = y * cpu_ops.sigmoid(y)
+        dt = dt + w("dt_bias")
+        step = (np.maximum(dt, 0) + np.log1p(np.exp(-np.abs(dt)))).astype(np.float32)
+        BC = np.repeat(y[:, inner:].reshape(T, 2, G, N), H // G, axis=2)
+        o = cpu_ops.state_space_recurrence(y[:, :inner].reshape(T, H, P), BC[:, 0], BC[:, 1], step, -np.exp(w("A_log")), w("D"), S)
+        o = (o.reshape(T, inner) * (z * cpu_ops.sigmoid(z))).reshape(T, a["norm_groups"], -1)
+        o = cpu_ops.rms_norm(o, np.ones(o.shape[-1], dtype=np.float32), a["eps"]).reshape(T, inner) * w("norm")
+        return cpu_ops.linear(o, w("o")) * np.float32(a.get("out_scale", 1.0))
 
     def _min_gru(self, p: PartSpec, x, store: dict, key):
         a = p.params
@@ -259,6 +282,10 @@ class CpuModel:
         return cpu_ops.linear(o, w("o"))
 
     def _mixer_of(self, part: PartSpec, h, positions, store, key):
+        if part.kind == "state_space":
+            return self._state_space(part, h, store, key)
+        if part.kind == "windowed_sink_attention":
+            return self._sink_attention(part, h, positions, store, key, None)
         if part.kind == "differential_attention":
             return self._differential(part, h, positions, store, key)
         if part.kind == "pooled_window_attention":
@@ -267,6 +294,8 @@ class CpuModel:
             return self._lightning(part, h, store, key)
         a = part.params                                            # parallel_mixers
         outs = [self._mixer_of(b["part"], h, positions, store, (key, i)) for i, b in enumerate(a["branches"])]
+        if a.get("combine") == "sum":
+            return sum(outs)
         ws = [self.w[part.tensor_name(b["out"])] for b in a["branches"]]
         return sum(cpu_ops.rms_norm(o, w, a["eps"]) for o, w in zip(outs, ws)) * np.float32(1.0 / len(outs))
 
@@ -275,6 +304,8 @@ class CpuModel:
         kind = sub.part.kind
         if kind in ("differential_attention", "pooled_window_attention", "lightning_attention", "parallel_mixers"):
             return self._mixer_of(sub.part, h, positions, store, m)
+        if kind == "state_space":
+            return self._state_space(sub.part, h, store, m)
         if kind == "channel_delta_rule":
             return self._delta_rule(sub.part, h, store, m)
         if kind == "gated_linear_attention":
@@ -318,14 +349,29 @@ class CpuModel:
         pos = a.get("position")
         rot = lambda t: t
         if pos is not None:
-            rot = lambda t: cpu_ops.rope_leading(t, positions, pos.params["dims"], pos.params["base"], pos.params.get("wave"))
-        q = rot(cpu_ops.linear(x, self.w[p.tensor_name(n["q"])]).reshape(T, nh, dk))
+            if pos.params.get("factor", 1.0) != 1.0:
+                rot = lambda t: cpu_ops.rotate_pairs(t, positions, pos.params["dims"], pos.params["base"], pos.params["factor"])
+            else:
+                rot = lambda t: cpu_ops.rope_leading(t, positions, pos.params["dims"], pos.params["base"], pos.params.get("wave"))
+        q = cpu_ops.linear(x, self.w[p.tensor_name(n["q"])])
+        keys_are_values = a.get("values") == "keys"
+        if keys_are_values:
+            raw = np.concatenate([q, cpu_ops.linear(x, self.w[p.tensor_name(n["k"])])], axis=1)
+            if a.get("conv"):
+                conv = np.concatenate([self.w[p.tensor_name(n[t] + a.get("conv_suffix", ".conv"))] for t in ("q", "k")]).astype(np.float32)
+                last = store.get((key, "conv"), np.zeros((a["conv"] - 1, raw.shape[1]), dtype=np.float32))
+                raw, store[(key, "conv")] = cpu_ops.causal_conv(raw, conv, last)
+            q, k = raw[:, :nh * dk], raw[:, nh * dk:].reshape(T, nkvh, dk)
+        q = rot(q.reshape(T, nh, dk))
         if a.get("q_temp"):
             q = q * cpu_ops.query_temperature(positions, a["q_temp"]["coef"], a["q_temp"]["every"])[:, None, None]
         bias = (self.w[p.tensor_name(n["r1"])], self.w[p.tensor_name(n["r2"])]) if a.get("distance_bias") else None
         if owner is None:
-            k = rot(cpu_ops.linear(x, self.w[p.tensor_name(n["k"])]).reshape(T, nkvh, dk))
-            v = cpu_ops.linear(x, self.w[p.tensor_name(n["v"])]).reshape(T, nkvh, dv)
+            if keys_are_values:
+                k, v = rot(k), k * np.float32(a.get("value_scale", 1.0))
+            else:
+                k = rot(cpu_ops.linear(x, self.w[p.tensor_name(n["k"])]).reshape(T, nkvh, dk))
+                v = cpu_ops.linear(x, self.w[p.tensor_name(n["v"])]).reshape(T, nkvh, dv)
             old = store.get(key)
             store[key] = (k, v) if old is None else (np.concatenate([old[0], k]), np.concatenate([old[1], v]))
             ks, vs = store[key]
@@ -344,7 +390,10 @@ class CpuModel:
              "shared_up": "shared.up", "shared_down": "shared.down", "shared_gate": "shared.sg", **(a.get("names") or {})}
         bias = self.w[p.tensor_name(n["bias"])] if a.get("use_bias", True) else None
         logits = cpu_ops.linear(x, self.w[p.tensor_name(n["router"])])
-        if a.get("groups") or a.get("renorm"):
+        if a.get("gate") == "softmax":
+            g = a.get("groups")
+            idx, wgt = cpu_ops.route_softmax(logits, bias, a["top"], (g["count"], g["keep"]) if g else None, a.get("route_scale", 1.0))
+        elif a.get("groups") or a.get("renorm"):
             g = a.get("groups")
             idx, wgt = cpu_ops.route_grouped(logits, a["top"], (g["count"], g["keep"]) if g else None, bool(a.get("renorm")),
                                              a.get("route_scale", 1.0))
@@ -352,15 +401,19 @@ class CpuModel:
             top_of = cpu_ops.route_top_softmax if a.get("gate") == "softmax_chosen" else cpu_ops.route_top
             idx, wgt = top_of(logits, bias, a["top"], a.get("route_scale", 1.0))
         act = cpu_ops.gelu if a.get("act") == "gelu" else cpu_ops.relu_squared
-        gated = a.get("act") == "swish_clamped"
+        gated = a.get("act") in ("swish_clamped", "silu")
         out = np.zeros((x.shape[0], a["hidden_size"]), dtype=np.float32)
         for t in range(x.shape[0]):
             for e, wt in zip(idx[t], wgt[t]):
+                if e >= a["experts"]:                              # an identity expert
+                    out[t] += wt * x[t]
+                    continue
                 up = self.w[p.tensor_name(n["expert_up"].format(e=int(e)))]
                 down = self.w[p.tensor_name(n["expert_down"].format(e=int(e)))]
                 if gated:
                     gate = self.w[p.tensor_name(n.get("expert_gate", "e{e}.gate").format(e=int(e)))]
-                    y = cpu_ops.swish_clamped(cpu_ops.linear(x[t:t + 1], gate), cpu_ops.linear(x[t:t + 1], up), a["limit"], a.get("alpha", 1.0))
+                    g1, u1 = cpu_ops.linear(x[t:t + 1], gate), cpu_ops.linear(x[t:t + 1], up)
+                    y = cpu_ops.glu(g1, u1, "silu") if a["act"] == "silu" else cpu_ops.swish_clamped(g1, u1, a["limit"], a.get("alpha", 1.0))
                 else:
                     y = act(cpu_ops.linear(x[t:t + 1], up))
                 out[t] += wt * cpu_ops.linear(y, down)[0]
@@ -443,7 +496,9 @@ class CpuModel:
         x = self._norm(self.spec.final_norm, x)
         head = self.spec.head
         name = head.params.get("tied_to") or head.tensor_name(head.params.get("tensor", "weight"))
-        return cpu_ops.linear(x, self.w[name]) * np.float32(head.params.get("scale", 1.0))
+        z = cpu_ops.linear(x, self.w[name]) * np.float32(head.params.get("scale", 1.0))
+        cap = np.float32(head.params.get("softcap") or 0.0)
+        return cap * np.tanh(z / cap) if cap else z
 
     def generate(self, prompt: Sequence[int], max_new_tokens: int, stop_ids: Sequence[int] = ()) -> List[int]:
         """Greedy continuation: the new tokens (a stop token included)."""

@@ -76,7 +76,8 @@ class LMHead(Part):
     """logits = h W^T in float32, no bias (xsmccc/llaisys src/models/qwen2/qwen2.cpp:76-77).
     With params["tied_to"] set, W is the tensor of that name (the embedding table) and the part
     declares no tensor of its own.  params: vocab_size, hidden_size, tied_to, tensor (the matrix's local name,
-    "weight" unless given), scale (default 1: the float32 logits are multiplied by it)."""
+    "weight" unless given), scale (default 1: the float32 logits are multiplied by it), softcap (default none: with a cap c > 0
+    the scaled logits z become c tanh(z / c))."""
     capturable = True
 
 
@@ -86,6 +87,9 @@ class LMHead(Part):
         self.tied_to = spec.params.get("tied_to")
         self.tensor = str(spec.params.get("tensor", "weight"))
         self.scale = float(spec.params.get("scale", 1.0))
+        self.softcap = float(spec.params.get("softcap") or 0.0)
+        if self.softcap < 0:
+            raise ValueError(f"a cap on the logits is positive, got {self.softcap}")
         self.weight = None
 
     def tensors(self):
@@ -101,4 +105,6 @@ class LMHead(Part):
     def forward(self, h):
         import torch
         logits = kernels.linear(h, self.weight, out_dtype=torch.float32)
-        return kernels.scale_(logits, self.scale) if self.scale != 1.0 else logits
+        if self.scale != 1.0:
+            kernels.scale_(logits, self.scale)
+        return kernels.softcap_(logits, self.softcap) if self.softcap else logits

@@ -54,7 +54,7 @@ class GatedMLP(FeedForward):
     """down(act(gate(x)) * up(x)) with the activation a parameter: "silu", "relu", "gelu_tanh", or "swish_clamped":
     g = min(gate(x), limit), u = clamp(up(x), -limit, limit), down(g sigmoid(alpha g) (u + 1)).  The gate
     and up matrices are kept as one [2I, H] matrix so that one product serves both; the activation and the product of
-    the halves are one pass in float32, or (silu and swish_clamped without biases) the epilogue of that product; a few tokens run in one launch.  With `bias` every projection has a bias (tensors named after the matrices with
+    the halves are one pass in float32, or (silu, relu and swish_clamped without biases) the epilogue of that product; a few tokens run in one launch.  With `bias` every projection has a bias (tensors named after the matrices with
     `bias_suffix`, default ".b").  The result is returned in float32 (it may be normed or scaled before it joins the
     stream) unless the part is asked to add it to the stream itself.  params: hidden_size, intermediate_size, act, limit and alpha (swish_clamped), bias, bias_suffix, names (local tensor names of gate, up, down)."""
     capturable = True
@@ -70,10 +70,10 @@ class GatedMLP(FeedForward):
             raise ValueError(f"the limit must be positive, got {self.limit}")
         self.names = dict({"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}, **(p.get("names") or {}))
         self.bias, self.bias_suffix = bool(p.get("bias", False)), str(p.get("bias_suffix", ".b"))
-        # what the products' own epilogues can do: no bias, and a sigmoid gate
+        # what the products' own epilogues can do: no bias, and a gate of that form
         self.form = None
-        if not self.bias and self.act in ("silu", "swish_clamped"):
-            self.form = kernels.GluForm() if self.act == "silu" else kernels.GluForm(self.limit, self.alpha, 1.0)
+        if not self.bias and self.act in ("silu", "relu", "swish_clamped"):
+            self.form = {"silu": kernels.GluForm(), "relu": kernels.RELU_GLU}.get(self.act) or kernels.GluForm(self.limit, self.alpha, 1.0)
         self.gate_up = self.down = self.b_gate_up = self.b_down = None
 
     def tensors(self):

@@ -29,6 +29,11 @@ class RoutedExperts(FeedForward):
     sigmoid(w_sg . h), one number per token (tensor `shared_gate`, [1, hidden]); its logit rides on the router's
     product as one more row of the matrix.
 
+    `gate` "softmax": gates are the softmax over all of the router's logits.  `group_score` "max": a group's score is its largest
+    choice score.  `identity` n: the router has n more outputs behind the experts', identity experts: they take part in the
+    softmax, the groups and the choice like the others, have no tensors, and a chosen one adds weight * h.  `act` "silu": a gated
+    expert, Wd (silu(Wg h) * Wu h).
+
     The experts' matrices are kept stacked ([E, ff, H] and [E, H, ff]).  A step's (token, choice) pairs are grouped by
     expert on the device (kernels.moe_plan) and the two products run over those groups: in bfloat16 on tcgen05, the
     second one ending in the weighted add into the float32 residual stream (float32 atomics, arrival order); in float32
@@ -38,7 +43,8 @@ class RoutedExperts(FeedForward):
     forward_into(..., scale=c) adds c times the part's output (the weights and the shared expert's activations carry the
     factor), for arrangements whose parts join the stream scaled.
 
-    params: hidden_size, experts, top, expert_ff, route_scale, gate, act, limit, alpha, groups, renorm, shared_ff (None: no
+    params: hidden_size, experts, top, expert_ff, route_scale, gate, act, limit, alpha, groups, group_score ("top2"
+    or "max"), renorm, identity, shared_ff (None: no
     shared expert), shared_gate, use_bias, names (local tensor names: router, bias, expert_up, expert_down with {e} for the expert's index, shared_up,
     shared_down, shared_gate).
     """
@@ -54,23 +60,28 @@ class RoutedExperts(FeedForward):
         self.ff = int(p["expert_ff"])
         self.route_scale = float(p.get("route_scale", 1.0))
         self.act = str(p.get("act", "relu_squared"))
-        if self.act not in ("relu_squared", "gelu", "swish_clamped"):
-            raise ValueError(f"expert activation {self.act!r} is not built (relu_squared, gelu, swish_clamped)")
-        self.gated = self.act == "swish_clamped"
+        if self.act not in ("relu_squared", "gelu", "swish_clamped", "silu"):
+            raise ValueError(f"expert activation {self.act!r} is not built (relu_squared, gelu, swish_clamped, silu)")
+        self.gated = self.act in ("swish_clamped", "silu")
         self.limit, self.alpha = float(p.get("limit", 0.0)), float(p.get("alpha", 1.0))
-        if self.gated and self.limit <= 0:
+        if self.act == "swish_clamped" and self.limit <= 0:
             raise ValueError(f"the clamped activation needs a positive limit, got {self.limit}")
         self.groups = (int(p["groups"]["count"]), int(p["groups"]["keep"])) if p.get("groups") else None
         self.renorm = bool(p.get("renorm", False))
         self.gate = str(p.get("gate", "sigmoid"))
         if self.gate not in kernels.ops.MOE_GATES:
             raise ValueError(f"unknown router gate {self.gate!r}; known: {sorted(kernels.ops.MOE_GATES)}")
-        if not (1 <= self.top <= self.n_experts):
-            raise ValueError(f"a token cannot use {self.top} of {self.n_experts} experts")
+        self.identity = int(p.get("identity") or 0)
+        self.n_outputs = self.n_experts + self.identity              # what the router chooses from
+        if self.identity < 0 or (self.identity and (self.gate == "softmax_chosen" or self.renorm)):
+            raise ValueError("identity experts go with gates that are not renormalised")
+        if not (1 <= self.top <= self.n_outputs):
+            raise ValueError(f"a token cannot use {self.top} of {self.n_outputs} experts")
+        self.group_max = {"top2": False, "max": True}[p.get("group_score", "top2")]
         if self.groups:
             count, keep = self.groups
-            if count < 1 or self.n_experts % count or not (1 <= keep <= count) or keep * (self.n_experts // count) < self.top:
-                raise ValueError(f"{self.n_experts} experts in {count} groups of which {keep} are kept cannot give {self.top} choices")
+            if count < 1 or self.n_outputs % count or not (1 <= keep <= count) or keep * (self.n_outputs // count) < self.top:
+                raise ValueError(f"{self.n_outputs} experts in {count} groups of which {keep} are kept cannot give {self.top} choices")
             if count == 1:
                 self.groups = None
         self.shared_ff = int(p["shared_ff"]) if p.get("shared_ff") else None
@@ -81,9 +92,9 @@ class RoutedExperts(FeedForward):
 
     def tensors(self):
         n = self.names
-        t = {n["router"]: TensorDecl((self.n_experts, self.hidden))}
+        t = {n["router"]: TensorDecl((self.n_outputs, self.hidden))}
         if self.use_bias:
-            t[n["bias"]] = TensorDecl((self.n_experts,), use="vector")
+            t[n["bias"]] = TensorDecl((self.n_outputs,), use="vector")
         for e in range(self.n_experts):
             t[n["expert_up"].format(e=e)] = TensorDecl((self.ff, self.hidden))
             if self.gated:
@@ -116,13 +127,22 @@ class RoutedExperts(FeedForward):
             self.shared_up, self.shared_down = tensors[n["shared_up"]].contiguous(), tensors[n["shared_down"]].contiguous()
 
     def forward(self, x, ctx):
-        out = torch.zeros((x.shape[0], self.hidden), dtype=torch.float32, device=x.device)
-        self.forward_into(x, ctx, out)
-        return out
+        return self._run(x, None, 1.0)
 
     def forward_into(self, x, ctx, residual, scale: float = 1.0):
-        idx, wgt, z = kernels.moe_route(x, self.router, self.bias, self.top, self.route_scale * scale, gate=self.gate,
-                                        n_experts=self.n_experts, with_logits=True, groups=self.groups, renorm=self.renorm)
+        self._run(x, residual, scale)
+        return True
+
+    def _run(self, x, residual, scale):
+        """The weighted sum added to `residual`, or (None) to a new float32 tensor; returns it."""
+        routed = kernels.moe_route(x, self.router, self.bias, self.top, self.route_scale * scale, gate=self.gate,
+                                   n_experts=self.n_outputs, with_logits=True, groups=self.groups, renorm=self.renorm,
+                                   group_max=self.group_max, identity=self.identity)
+        idx, wgt, z = routed[:3]
+        if self.identity:
+            residual = kernels.moe_identity(x, routed[3], residual)
+        elif residual is None:
+            residual = torch.zeros((x.shape[0], self.hidden), dtype=torch.float32, device=x.device)
         tc = kernels.moe_tc_ok(x, self.up, self.down) and residual.stride(1) == 1
         plan = kernels.moe_plan(idx, self.n_experts, kernels.moe_tc_tile_rows(idx.numel(), self.n_experts) if tc else None)
         if tc:
@@ -142,11 +162,11 @@ class RoutedExperts(FeedForward):
         if self.shared_ff:
             a = kernels.linear(x, self.shared_up)
             if self.shared_gate or scale != 1.0 or self.act != "relu_squared":
-                kernels.act_rows_(a, self.act, z[:, self.n_experts] if self.shared_gate else None, scale)
+                kernels.act_rows_(a, self.act, z[:, self.n_outputs] if self.shared_gate else None, scale)
             else:
                 kernels.relu_squared_(a)
             if kernels.linear_into_ok(a, self.shared_down, None, residual):
                 kernels.linear_into(a, self.shared_down, None, residual)
             else:
                 kernels.residual_add(residual, kernels.linear(a, self.shared_down))
-        return True
+        return residual

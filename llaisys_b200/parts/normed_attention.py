@@ -288,18 +288,22 @@ class LightningAttention(Mixer):
 @register_part("mixer", "parallel_mixers")
 class ParallelMixers(Mixer):
     """Several mixers side by side that read the same input; the result is the mean of their outputs, each first
-    RMS-normed over the model width with a weight of its own.  The branches are mixers of any kind, built from their
+    RMS-normed over the model width with a weight of its own, or, with combine "sum", the sum of their outputs (each branch
+    brings a constant of its own as part of its spec).  The branches are mixers of any kind, built from their
     own specs (their tensors lie under their own prefixes); their users of the cache follow one another.
 
-    params: hidden_size, eps, branches: [{part: PartSpec of category "mixer", out: the local name of the branch's norm
-    weight}]."""
+    A sum is formed by the branches' own last kernels where they can (forward_into), in float32.
+
+    params: hidden_size, eps, combine ("normed_mean" unless given, or "sum"), branches: [{part: PartSpec of category "mixer", out:
+    the local name of the branch's norm weight (normed_mean)}]."""
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
         p = spec.params
-        self.hidden, self.eps = int(p["hidden_size"]), float(p["eps"])
+        self.hidden, self.eps = int(p["hidden_size"]), float(p.get("eps", 0.0))
+        self.sum = {"normed_mean": False, "sum": True}[p.get("combine", "normed_mean")]
         self.branches = [build_part("mixer", b["part"], env) for b in p["branches"]]
-        self.out_names = [str(b["out"]) for b in p["branches"]]
+        self.out_names = [] if self.sum else [str(b["out"]) for b in p["branches"]]
         if not (1 <= len(self.branches) <= 4):
             raise ValueError(f"one to four branches, got {len(self.branches)}")
         self.out_w = []
@@ -324,7 +328,32 @@ class ParallelMixers(Mixer):
     def load(self, tensors):
         self.out_w = [tensors[n].float().contiguous() for n in self.out_names]
 
+    def forward_into(self, x, ctx, call, residual):
+        if not self.sum:
+            return False
+        for b in self.branches:
+            if not b.forward_into(x, ctx, call, residual):
+                kernels.residual_add(residual, b.forward(x, ctx, call))
+            call += len(b.cache_users())
+        return True
+
     def forward(self, x, ctx, call):
+        if self.sum and (x.shape[0] > 256 or len(self.branches) == 1):
+            # many tokens: every branch's product adds into one buffer (the first one's too: the paired-SM kernel adds, or rounds)
+            out = torch.zeros((x.shape[0], self.hidden), dtype=torch.float32, device=x.device)
+            self.forward_into(x, ctx, call, out)
+            return out
+        if self.sum:
+            out = None
+            for b in self.branches:
+                if out is None or not b.forward_into(x, ctx, call, out):
+                    y = b.forward(x, ctx, call)
+                    if out is None:
+                        out = y if y.dtype == torch.float32 else y.float()
+                    else:
+                        kernels.residual_add(out, y)
+                call += len(b.cache_users())
+            return out
         outs = []
         for b in self.branches:
             y = b.forward(x, ctx, call)

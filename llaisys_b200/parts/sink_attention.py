@@ -25,7 +25,12 @@ class WindowedSinkAttention(Mixer):
       * a query temperature (`q_temp` = {coef, every}): the query at position p is multiplied by
         1 + coef ln(floor((p + 1) / every) + 1), i.e. queries sharpen as the sequence grows, in steps of `every`;
       * a layer without key and value projections (`own_kv` false) that reads the rotated keys and the values another
-        layer stored in the cache (the run order's `cache_of`), with queries, window and everything else its own.
+        layer stored in the cache (the run order's `cache_of`), with queries, window and everything else its own;
+      * values that are the keys (`values` "keys"): a value head is its key head before the rotation, there is no value projection;
+        queries and keys may then pass a causal convolution of `conv` tokens per channel first (tensors named after their
+        projections with `conv_suffix`; the last conv - 1 inputs are a second user of the cache, a fixed-size state);
+      * values times a constant (`value_scale`, with values "keys"), i.e. the part's output times it; an output that is float32 in
+        both precisions (`out_f32`).
 
     Query heads h of a group of num_heads / num_kv_heads share key/value head h / group.  Scores are (q . k) * scale.
     The position encoding is a part of category "position" that hands out leading_tables() (rotation of a head's
@@ -38,7 +43,7 @@ class WindowedSinkAttention(Mixer):
     otherwise (and in decode) keys and values are appended first and attention reads the cache alone.
 
     params: hidden_size, num_heads, num_kv_heads, key_dim, value_dim, scale, window, keep_first, sink, own_kv,
-    cache_window, position (PartSpec or None: no rotation), distance_bias, q_temp, softcap, gate, names (local tensor names of
+    cache_window, position (PartSpec or None: no rotation), distance_bias, q_temp, softcap, gate, values, conv, conv_suffix, value_scale, out_f32, names (local tensor names of
     q, k, v, o, r1, r2, sink, g; default those).
     """
 
@@ -79,7 +84,16 @@ class WindowedSinkAttention(Mixer):
             self.q_temp = (float(p["q_temp"]["coef"]), int(p["q_temp"]["every"]))
             if self.q_temp[1] <= 0:
                 raise ValueError(f"the query temperature's period must be positive, got {self.q_temp[1]}")
-        self.w_in = self.w_o = self.r1 = self.r2 = self.sink_logits = None
+        if p.get("values", "own") not in ("own", "keys"):
+            raise ValueError(f"values are the layer's 'own' or its 'keys', got {p['values']!r}")
+        self.keys_are_values = p.get("values") == "keys"
+        self.taps, self.conv_suffix = int(p.get("conv") or 1), str(p.get("conv_suffix", ".conv"))
+        self.value_scale, self.out_f32 = float(p.get("value_scale", 1.0)), bool(p.get("out_f32", False))
+        if self.keys_are_values and (not self.own_kv or self.dk != self.dv):
+            raise ValueError("values that are the keys need key projections of the layer's own and one width")
+        if not self.keys_are_values and (p.get("conv") or self.value_scale != 1.0):
+            raise ValueError("the convolution and the values' constant are built for values that are the keys")
+        self.w_in = self.w_o = self.r1 = self.r2 = self.sink_logits = self.conv = None
 
     capturable = True
 
@@ -90,12 +104,20 @@ class WindowedSinkAttention(Mixer):
     def kv_need(self):
         return KVNeed(self.nkvh, self.dk, self.dv, self.cache_window, self.keep_first if self.cache_window is not None else 0)
 
+    def cache_users(self):
+        state = (self.taps - 1) * (self.nh + self.nkvh) * self.dk
+        return [(self.kv_need(), 0)] + ([(None, state)] if state else [])
+
     def tensors(self):
         n = self.names
         t = {n["q"]: TensorDecl((self.nh * self.dk, self.hidden)), n["o"]: TensorDecl((self.hidden, self.nh * self.dv))}
         if self.own_kv:
             t[n["k"]] = TensorDecl((self.nkvh * self.dk, self.hidden))
-            t[n["v"]] = TensorDecl((self.nkvh * self.dv, self.hidden))
+            if not self.keys_are_values:
+                t[n["v"]] = TensorDecl((self.nkvh * self.dv, self.hidden))
+        if self.taps > 1 or self.spec.params.get("conv"):
+            for k, heads in (("q", self.nh), ("k", self.nkvh)):
+                t[n[k] + self.conv_suffix] = TensorDecl((heads * self.dk, self.taps), init="mean:0.25", use="vector")
         if self.learned_sink:
             t[n["sink"]] = TensorDecl((self.nh,), use="vector")
         if self.gated:
@@ -107,20 +129,26 @@ class WindowedSinkAttention(Mixer):
 
     def load(self, tensors):
         n = self.names
-        ts = [tensors[n["q"]]] + ([tensors[n["k"]], tensors[n["v"]]] if self.own_kv else []) + ([tensors[n["g"]]] if self.gated else [])
+        kv = ("k",) if self.keys_are_values else ("k", "v") if self.own_kv else ()
+        ts = [tensors[n["q"]]] + [tensors[n[k]] for k in kv] + ([tensors[n["g"]]] if self.gated else [])
         dt = ts[0].dtype
         for t in ts[1:]:
             dt = torch.promote_types(dt, t.dtype)
         self.w_in = torch.cat([t.to(dt) for t in ts], dim=0).contiguous()
         self.w_o = tensors[n["o"]].contiguous()
         self.gate_off = self.w_in.shape[0] - self.nh * self.dv              # the gate's columns, when there is one
+        if self.keys_are_values:
+            rows = (self.nh + self.nkvh) * self.dk
+            self.conv = torch.ones((1, rows), dtype=torch.float32, device=self.w_in.device)
+            if self.spec.params.get("conv"):
+                self.conv = torch.cat([tensors[n[k] + self.conv_suffix].float() for k in ("q", "k")], dim=0).t().contiguous()   # [taps, channels]
         if self.learned_sink:
             self.sink_logits = tensors[n["sink"]].float().contiguous()
         if self.distance_bias:
             self.r1, self.r2 = tensors[n["r1"]].float().contiguous(), tensors[n["r2"]].float().contiguous()
 
     def forward(self, x, ctx, call):
-        return kernels.linear(self._attend(x, ctx, call), self.w_o)
+        return kernels.linear(self._attend(x, ctx, call), self.w_o, out_dtype=torch.float32 if self.out_f32 else None)
 
     def forward_into(self, x, ctx, call, residual):
         if not (x.dtype == torch.bfloat16 and self.w_o.dtype == torch.bfloat16
@@ -160,17 +188,24 @@ class WindowedSinkAttention(Mixer):
         extras = kernels.AttnExtras(value_dim=self.dv, keep_first=self.keep_first, pinned=kv.pinned, sink=self.sink,
                                     sink_logits=self.sink_logits, softcap=self.softcap,
                                     dist_bias=(self.r1, self.r2) if self.distance_bias else None, q_temp=self.q_temp)
+        ring_cache = kv.writable and self.cache_window is not None
+        prepared = self.keys_are_values
+        if prepared:
+            proj = kernels.conv_heads(proj[:, :(self.nh + self.nkvh) * self.dk], self.nh, self.nkvh, self.dk, self.conv,
+                                      ctx.state(call + 1) if self.taps > 1 else None, ctx, (cos, sin, self.rot) if cos is not None else None,
+                                      self.value_scale, append if ctx.is_decode or not ring_cache else None)
         common = (proj, self.nh, self.nkvh, self.dk, kv.k, kv.v, kv.page_table, kv.ring, ctx.seq_start, ctx.seq_len_before,
                   ctx.n_seqs)
-        ring_cache = kv.writable and self.cache_window is not None
         if ctx.is_decode or not ring_cache:
-            kernels.rope_lead_append(proj, self.nh, nkv_here, self.dk, self.dv, self.rot, cos=cos, sin=sin,
-                                     tok_pos=ctx.tok_pos, append=append, err=ctx.err)
+            if not prepared:
+                kernels.rope_lead_append(proj, self.nh, nkv_here, self.dk, self.dv, self.rot, cos=cos, sin=sin,
+                                         tok_pos=ctx.tok_pos, append=append, err=ctx.err)
             if ctx.is_decode:
                 return kernels.attention_decode(*common, self.window, self.scale, n_splits=self._splits(ctx), extras=extras)
             return kernels.attention_prefill(*common, ctx.max_new, self.window, self.scale, all_from_cache=True, extras=extras)
-        kernels.rope_lead_append(proj, self.nh, nkv_here, self.dk, self.dv, self.rot, cos=cos, sin=sin,
-                                 tok_pos=ctx.tok_pos, err=ctx.err)
+        if not prepared:
+            kernels.rope_lead_append(proj, self.nh, nkv_here, self.dk, self.dv, self.rot, cos=cos, sin=sin,
+                                     tok_pos=ctx.tok_pos, err=ctx.err)
         out = kernels.attention_prefill(*common, ctx.max_new, self.window, self.scale, all_from_cache=False, extras=extras)
         kernels.rope_lead_append(proj, self.nh, nkv_here, self.dk, self.dv, 0, tok_pos=ctx.tok_pos, append=append, err=ctx.err)
         return out
