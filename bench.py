@@ -633,14 +633,37 @@ def bezadra_configs(size: str, layers: int):
     return bz, nubedra_configs(size, layers)[0]
 
 
+def zupitar_configs(size: str, layers: int):
+    """(Zupitar config, Zetalorn config) of one size: the same width, heads, head size and routed experts as the Zetalorn model of
+    that size (here with eight identity experts behind them).  Layers in turn: a parallel one (attention beside a state-space mixer
+    as wide as the stream) with routed experts, and a state-space one twice as wide with a dense feed-forward that is as wide as the
+    experts a token uses.  State-space heads have 64 value channels and 128 state rows, in four groups."""
+    D, H, G, dh, rot, _, _, E, top, ff, _ = DESIGN_SIZES[size]
+
+    def mamba(inner):
+        return {"heads": inner // 64, "vdim": 64, "state": 128, "groups": 4, "conv": 4, "norm_groups": 4}
+
+    kinds = [
+        {"type": "parallel", "mixer": {
+            "left": {"heads": H, "kv_heads": G, "dim": dh, "vdim": dh, "scale": dh ** -0.5, "conv": 4,
+                     "rot": {"dims": rot, "base": 1000000.0, "scaling": {"factor": 4.0}}},
+            "right": mamba(D), "left_scale": 1.1, "right_scale": 0.8},
+         "mlp": {"kind": "moe", "router": {"experts": E, "top": top, "identity": 8, "groups": {"count": 8, "keep": 4}}, "expert": {"ff": ff}}},
+        {"type": "mamba2", "mixer": mamba(2 * D), "mlp": {"kind": "dense", "ff": top * ff}},
+    ]
+    zu = {"architecture": "Zupitar", "vocab": 32768, "width": D, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+          "layers": [kinds[i % 2] for i in range(layers)]}
+    return zu, zetalorn_configs(size, layers)[0]
+
+
 DESIGNS = {"vumezen": (DESIGN_SIZES, design_configs, "qwen2"), "nubedra": (NUBEDRA_SIZES, nubedra_configs, "qwen2"),
            "zedirax": (NUBEDRA_SIZES, zedirax_configs, "nubedra"), "zetalorn": (DESIGN_SIZES, zetalorn_configs, "vumezen"),
-           "bezadra": (NUBEDRA_SIZES, bezadra_configs, "nubedra")}
+           "bezadra": (NUBEDRA_SIZES, bezadra_configs, "nubedra"), "zupitar": (DESIGN_SIZES, zupitar_configs, "zetalorn")}
 
 
 def design_run(args) -> int:
     """Prefill (one step over --tokens tokens) and decode (--batch sequences that hold --tokens tokens each) of the
-    chosen design and of the model beside it (the Qwen2 dense decoder; for zedirax and bezadra the Nubedra design, for zetalorn the Vumezen design) at equal layer sizes: time per step, tokens a second, and each kernel's
+    chosen design and of the model beside it (the Qwen2 dense decoder; for zedirax and bezadra the Nubedra design, for zetalorn the Vumezen design, for zupitar the Zetalorn design) at equal layer sizes: time per step, tokens a second, and each kernel's
     share of a step (torch.profiler).  One JSON line per model and phase.  Inputs: the weights of either model are
     larger than L2, and nothing is flushed between steps."""
     import collections
@@ -875,7 +898,7 @@ def main() -> int:
     ap.add_argument("--timeline", choices=["decode", "prefill"], default=None,
                     help="print the per-kernel timeline of a step (torch.profiler, no ncu) instead of measuring")
     ap.add_argument("--design", choices=sorted(DESIGNS), default=None,
-                    help="measure this design beside the Qwen2 dense decoder (zedirax, bezadra: beside the Nubedra design; zetalorn: beside the Vumezen design) at equal layer sizes "
+                    help="measure this design beside the Qwen2 dense decoder (zedirax, bezadra: beside the Nubedra design; zetalorn: beside the Vumezen design; zupitar: beside the Zetalorn design) at equal layer sizes "
                          "(prefill of --tokens tokens, decode at --batch) instead of the benchmark; --size picks among the sizes "
                          "(default: all)")
     ap.add_argument("--size", default=None, help="with --design: comma-separated sizes of " + ", ".join(sorted(DESIGN_SIZES)))
