@@ -953,6 +953,89 @@ scaled_norm_add_kernel(float* __restrict__ residual, const TD* __restrict__ delt
         out[(size_t)r * H + j] = from_f32<TO>(rowbuf[j] * inv * (to_f32(w_next[j]) + offset));
 }
 
+// The same for rows of up to 8,192 elements in whole 16-byte pieces: the row stays in registers (PER pieces a thread), so every
+// input is read once and all of a thread's reads are under way together.
+template <typename T> __device__ __forceinline__ float4 load_four(const T* src);
+template <> __device__ __forceinline__ float4 load_four<float>(const float* src) { return *reinterpret_cast<const float4*>(src); }
+template <> __device__ __forceinline__ float4 load_four<bf16>(const bf16* src) {
+    const uint2 q = *reinterpret_cast<const uint2*>(src);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&q);
+    return make_float4(__low2float(h[0]), __high2float(h[0]), __low2float(h[1]), __high2float(h[1]));
+}
+__device__ __forceinline__ void store_four(float* dst, float4 v) { *reinterpret_cast<float4*>(dst) = v; }
+__device__ __forceinline__ void store_four(bf16* dst, float4 v) {
+    uint2 q;
+    *reinterpret_cast<__nv_bfloat162*>(&q.x) = __floats2bfloat162_rn(v.x, v.y);
+    *reinterpret_cast<__nv_bfloat162*>(&q.y) = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(dst) = q;
+}
+__device__ __forceinline__ float dot_self(float4 v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); }
+
+template <typename TD, typename TW, typename TO, int PER>
+__global__ void __launch_bounds__(256)
+scaled_norm_add_vec_kernel(float* __restrict__ residual, const TD* __restrict__ delta, const TW* __restrict__ w_post,
+                           float mult, const TW* __restrict__ w_next, TO* __restrict__ out, int H, float eps, float offset) {
+    __shared__ float red[2][8];
+    const int r = blockIdx.x, tid = threadIdx.x, lane = tid & 31, wp = tid >> 5;
+    float4 wn[PER], wq[PER];
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {                        // (weights: no kernel of a step writes them)
+        const int j = (tid + k * 256) * 4;
+        wq[k] = delta && j < H ? load_four<TW>(w_post + j) : zero;
+        wn[k] = out && j < H ? load_four<TW>(w_next + j) : zero;
+    }
+    llb_grid_dependency_sync();
+    float* res = residual + (size_t)r * H;
+    float4 x[PER], d[PER];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int j = (tid + k * 256) * 4;
+        d[k] = delta && j < H ? load_four<TD>(delta + (size_t)r * H + j) : zero;
+        x[k] = j < H ? load_four<float>(res + j) : zero;
+    }
+    if (delta) {
+#pragma unroll
+        for (int k = 0; k < PER; ++k) ss += dot_self(d[k]);
+        ss = warp_sum(ss);
+        if (lane == 0) red[0][wp] = ss;
+        __syncthreads();
+        float tot = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) tot += red[0][i];
+        const float inv = mult / sqrtf(tot / (float)H + eps);
+#pragma unroll
+        for (int k = 0; k < PER; ++k) {
+            const int j = (tid + k * 256) * 4;
+            x[k].x += d[k].x * inv * (wq[k].x + offset);
+            x[k].y += d[k].y * inv * (wq[k].y + offset);
+            x[k].z += d[k].z * inv * (wq[k].z + offset);
+            x[k].w += d[k].w * inv * (wq[k].w + offset);
+            if (j < H) store_four(res + j, x[k]);
+            else x[k] = zero;
+        }
+    }
+    if (!out) return;
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) ss += dot_self(x[k]);
+    ss = warp_sum(ss);
+    if (lane == 0) red[1][wp] = ss;
+    __syncthreads();
+    float tot = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) tot += red[1][i];
+    const float inv = 1.0f / sqrtf(tot / (float)H + eps);
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int j = (tid + k * 256) * 4;
+        if (j < H)
+            store_four(out + (size_t)r * H + j, make_float4(x[k].x * inv * (wn[k].x + offset), x[k].y * inv * (wn[k].y + offset),
+                                                            x[k].z * inv * (wn[k].z + offset), x[k].w * inv * (wn[k].w + offset)));
+    }
+}
+
 LLB_API int llb_scaled_norm_add(float* residual, const void* delta, int delta_dtype, const void* w_post, float mult,
                                 const void* w_next, int w_dtype, void* out, int out_dtype, int R, int H, float eps,
                                 float offset, cudaStream_t stream) {
@@ -964,6 +1047,14 @@ LLB_API int llb_scaled_norm_add(float* residual, const void* delta, int delta_dt
     LLB_DISPATCH_DTYPE(delta_dtype, TD, {
         LLB_DISPATCH_DTYPE(w_dtype, TW, {
             LLB_DISPATCH_DTYPE(out_dtype, TO, {
+                if (H % 4 == 0 && H <= 8192 &&
+                    !(((uintptr_t)residual | (uintptr_t)delta | (uintptr_t)w_post | (uintptr_t)w_next | (uintptr_t)out) & 15)) {
+                    auto v = H <= 1024 ? scaled_norm_add_vec_kernel<TD, TW, TO, 1> : H <= 2048 ? scaled_norm_add_vec_kernel<TD, TW, TO, 2>
+                           : H <= 4096 ? scaled_norm_add_vec_kernel<TD, TW, TO, 4> : scaled_norm_add_vec_kernel<TD, TW, TO, 8>;
+                    llb_launch(v, dim3(R), dim3(256), 0, stream, residual, (const TD*)delta, (const TW*)w_post, mult, (const TW*)w_next,
+                               (TO*)out, H, eps, offset);
+                    return llb_status();
+                }
                 auto k = scaled_norm_add_kernel<TD, TW, TO>;
                 if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
                 llb_launch(k, dim3(R), dim3(256), smem, stream, residual, (const TD*)delta, (const TW*)w_post, mult,

@@ -168,17 +168,22 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
     lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
-// [CHUNK rows, cols] of the operand from column c0 on into a tile of `pad` columns (a multiple of 16): 16-byte pieces where the
-// rows allow it; zeros beyond `cols` and beyond the chunk's tokens.
+// 16 bytes into shared memory without waiting for them (zeros unless `in`).
+__device__ __forceinline__ void copy16(bf16* dst, const bf16* src, bool in) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void copies_done() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
+// [CHUNK rows, cols] of the operand into a tile of `pad` columns (a multiple of 16): 16-byte asynchronous copies where the rows
+// allow it; zeros beyond `cols` and beyond the chunk's tokens.
 __device__ __forceinline__ void load_tile(bf16* dst, int dst_ld, const bf16* src, int ld, int rows, int cols, int pad, bool vec) {
     const int tid = threadIdx.x;
     if (vec) {
         const int per = pad / 8;
         for (int i = tid; i < CHUNK * per; i += CHUNK_THREADS) {
             const int r = i / per, c = (i - r * per) * 8;
-            uint4 q = make_uint4(0u, 0u, 0u, 0u);
-            if (r < rows && c < cols) q = *reinterpret_cast<const uint4*>(src + (size_t)r * ld + c);
-            *reinterpret_cast<uint4*>(dst + r * dst_ld + c) = q;
+            const bool in = r < rows && c < cols;
+            copy16(dst + r * dst_ld + c, in ? src + (size_t)r * ld + c : src, in);
         }
     } else {
         for (int i = tid; i < CHUNK * pad; i += CHUNK_THREADS) {
@@ -231,6 +236,17 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_state_kernel(SsdParam
     const int nc = min(CHUNK, n - c * CHUNK), row0 = tok0 + c * CHUNK;
     const bf16* src = (const bf16*)p.xbc + (size_t)row0 * p.ld;
     load_tile(sB, bld, src + inner + g * N, p.ld, nc, N, npad, vec);
+    // (the rows of x are under way before the decays are formed)
+    constexpr int XP = CHUNK * (PT / 8) / CHUNK_THREADS;
+    uint4 xq[XP];
+    if (vec) {
+#pragma unroll
+        for (int k = 0; k < XP; ++k) {
+            const int i = tid + k * CHUNK_THREADS, r = i / (PT / 8), cc = (i - r * (PT / 8)) * 8;
+            xq[k] = make_uint4(0u, 0u, 0u, 0u);
+            if (r < nc && p0 + cc < P) xq[k] = *reinterpret_cast<const uint4*>(src + h * P + p0 + (size_t)r * p.ld + cc);
+        }
+    }
     chunk_decays(p, row0, nc, h, scum, sdt);
     __syncthreads();
     const float end = scum[CHUNK - 1];
@@ -239,12 +255,12 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_state_kernel(SsdParam
     {
         const bf16* xs = src + h * P + p0;
         if (vec) {
-            for (int i = tid; i < CHUNK * (PT / 8); i += CHUNK_THREADS) {
-                const int r = i / (PT / 8), cc = (i - r * (PT / 8)) * 8;
-                uint4 q = make_uint4(0u, 0u, 0u, 0u), hi, lo;
-                if (r < nc && p0 + cc < P) q = *reinterpret_cast<const uint4*>(xs + (size_t)r * p.ld + cc);
+#pragma unroll
+            for (int k = 0; k < XP; ++k) {
+                const int i = tid + k * CHUNK_THREADS, r = i / (PT / 8), cc = (i - r * (PT / 8)) * 8;
+                uint4 hi, lo;
                 const float w = expf(end - scum[r]) * sdt[r];
-                const __nv_bfloat162* x2 = reinterpret_cast<const __nv_bfloat162*>(&q);
+                const __nv_bfloat162* x2 = reinterpret_cast<const __nv_bfloat162*>(&xq[k]);
                 uint32_t* h4 = reinterpret_cast<uint32_t*>(&hi);
                 uint32_t* l4 = reinterpret_cast<uint32_t*>(&lo);
 #pragma unroll
@@ -262,6 +278,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_state_kernel(SsdParam
             }
         }
     }
+    copies_done();
     __syncthreads();
     float* rec = p.rec + chunk * N * P;
     const uint32_t ab = smem_addr(sB) + (((lane & 7) + ((lane >> 4) << 3)) * bld + ((lane >> 3) & 1) * 8) * 2;
@@ -369,27 +386,37 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
     {
         const float* rec = p.rec + ((size_t)(chunk_base(tok0, b) + c) * p.H + h) * N * P + p0;
         const bool vec4 = P % 4 == 0;
-        for (int i = tid; i < npad * (PT / 4); i += CHUNK_THREADS) {
-            const int r = i / (PT / 4), cc = (i - r * (PT / 4)) * 4;
-            float4 q = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (r < N && p0 + cc < P) {
+        constexpr int AHEAD = 8;                           // pieces under way at a time
+        for (int i0 = tid; i0 < npad * (PT / 4); i0 += AHEAD * CHUNK_THREADS) {
+            float4 q[AHEAD];
+#pragma unroll
+            for (int k = 0; k < AHEAD; ++k) {
+                const int i = i0 + k * CHUNK_THREADS, r = i / (PT / 4), cc = (i - r * (PT / 4)) * 4;
+                q[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (r >= N || p0 + cc >= P) continue;
                 const float* s = rec + (size_t)r * P + cc;
-                if (vec4) q = *reinterpret_cast<const float4*>(s);
+                if (vec4) q[k] = *reinterpret_cast<const float4*>(s);
                 else {
-                    q.x = s[0];
-                    if (p0 + cc + 1 < P) q.y = s[1];
-                    if (p0 + cc + 2 < P) q.z = s[2];
-                    if (p0 + cc + 3 < P) q.w = s[3];
+                    q[k].x = s[0];
+                    if (p0 + cc + 1 < P) q[k].y = s[1];
+                    if (p0 + cc + 2 < P) q[k].z = s[2];
+                    if (p0 + cc + 3 < P) q[k].w = s[3];
                 }
             }
-            uint2 hi, lo;
-            split2(q.x, q.y, hi.x, lo.x);
-            split2(q.z, q.w, hi.y, lo.y);
-            *reinterpret_cast<uint2*>(sHi + r * PLD + cc) = hi;
-            *reinterpret_cast<uint2*>(sLo + r * PLD + cc) = lo;
+#pragma unroll
+            for (int k = 0; k < AHEAD; ++k) {
+                const int i = i0 + k * CHUNK_THREADS, r = i / (PT / 4), cc = (i - r * (PT / 4)) * 4;
+                if (r >= npad) break;
+                uint2 hi, lo;
+                split2(q[k].x, q[k].y, hi.x, lo.x);
+                split2(q[k].z, q[k].w, hi.y, lo.y);
+                *reinterpret_cast<uint2*>(sHi + r * PLD + cc) = hi;
+                *reinterpret_cast<uint2*>(sLo + r * PLD + cc) = lo;
+            }
         }
     }
     chunk_decays(p, row0, nc, h, scum, sdt);
+    copies_done();
     __syncthreads();
     const int t0 = warp * 16;
     if (t0 >= nc) return;                                  // (no barrier follows)

@@ -17,6 +17,8 @@ TEST_MODULES = [
     ("attention_simt.cu", {"LLB_HEAD_DIM": 12}),
     # capped scores with a learned sink (test_gpu_bezadra.py)
     ("attention_simt.cu", {"LLB_HEAD_DIM": 96}), ("attention_mma.cu", {"LLB_HEAD_DIM": 96}), ("attention_simt.cu", {"LLB_HEAD_DIM": 2, "LLB_VALUE_DIM": 1}),
+    # values that are the keys (test_gpu_zupitar.py)
+    *[("attention_simt.cu", {"LLB_HEAD_DIM": d}) for d in (2,)],
     # the build in which a bounded wait can be made to run out (test_gpu_kernels.py)
     ("gemm_tc.cu", {"LLB_WAIT_LIMIT": 4096, "LLB_TEST_STALL": 1}),
 ]
