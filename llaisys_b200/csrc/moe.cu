@@ -82,6 +82,7 @@ moe_select_kernel(const float* __restrict__ z, int ldz, const float* __restrict_
             if (gs[e / per] != INFINITY) choice[e] = -INFINITY;
         __syncwarp();
     }
+    float identity_sum = 0.f;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int arg = 0x7fffffff;
@@ -103,6 +104,7 @@ moe_select_kernel(const float* __restrict__ z, int ldz, const float* __restrict_
             idx[(size_t)t * top + k] = arg;
             wgt[(size_t)t * top + k] = mode == 1 ? gate[arg] : gate[arg] * route_scale;
             choice[arg] = -INFINITY;
+            if (arg >= E - identity) identity_sum += gate[arg] * route_scale;
         }
         __syncwarp();
     }
@@ -120,12 +122,7 @@ moe_select_kernel(const float* __restrict__ z, int ldz, const float* __restrict_
         const float inv = route_scale / sum;
         for (int k = 0; k < top; ++k) w[k] *= inv;
     }
-    if (identity_wgt && lane == 0) {
-        float sum = 0.f;
-        for (int k = 0; k < top; ++k)
-            if (idx[(size_t)t * top + k] >= E - identity) sum += wgt[(size_t)t * top + k];
-        identity_wgt[t] = sum;
-    }
+    if (identity_wgt && lane == 0) identity_wgt[t] = identity_sum;
     if (mode != 1 && renorm && lane == 0) {
         // the chosen gates divided by their sum (the factor route_scale is in them already)
         float* w = wgt + (size_t)t * top;

@@ -202,8 +202,9 @@ __global__ void __launch_bounds__(THREADS) conv_heads_kernel(ConvHeads p) {
     const int last = p.append ? p.seq_len_before[b] + n - 1 : 0, kvh = head - p.n_q;
     T* kpool = (T*)p.kpool;
     T* vpool = (T*)p.vpool;
+    const int pos0 = __ldg(p.tok_pos + tok0);              // (a sequence's tokens of a step stand at consecutive positions)
     conv_run<T, TAPS, 2, U>(p.conv, col, have, b, tok0, n, at0, [&](int t, float (&v)[2][U]) {
-        const int pos = p.tok_pos[tok0 + t];
+        const int pos = pos0 + t;
         if (p.rot > 0 && (pos < 0 || pos >= p.table_rows)) {
             atomicExch(p.err, 2);
             return;
@@ -225,7 +226,7 @@ __global__ void __launch_bounds__(THREADS) conv_heads_kernel(ConvHeads p) {
         if (pair) {
 #pragma unroll
             for (int e = 0; e < U; ++e) {
-                const float c = p.cos_t[(size_t)pos * half + first + e], s = p.sin_t[(size_t)pos * half + first + e];
+                const float c = __ldg(p.cos_t + (size_t)pos * half + first + e), s = __ldg(p.sin_t + (size_t)pos * half + first + e);
                 const float x0 = v[0][e], x1 = v[1][e];
                 v[0][e] = x0 * c - x1 * s;
                 v[1][e] = x1 * c + x0 * s;

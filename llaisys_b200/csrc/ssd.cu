@@ -34,6 +34,7 @@ struct SsdParams {
     int H, P, N, G;
     float* rec;               // [chunks, H, N P]: a chunk's own sum, then the state it starts with
     float* decay;             // [chunks, H]: exp(c_end)
+    float* sums;              // [chunks, H, 2 * 64]: c_t of the chunk's tokens, then their steps
 };
 
 __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
@@ -143,6 +144,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssd_scan_kernel(SsdParams p) {
 // ------------------------------------------------------------------ long steps, chunk by chunk
 constexpr int CHUNK = 64;
 constexpr int CHUNK_THREADS = 128;
+static_assert(CHUNK_THREADS == 2 * CHUNK, "a thread per number of a chunk's sums");
 constexpr int PT = 64;                  // value channels of a block
 constexpr int PLD = PT + 8;             // row stride of a tile of PT columns: rows 16 bytes apart modulo 128
 
@@ -252,6 +254,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_state_kernel(SsdParam
     const float end = scum[CHUNK - 1];
     const size_t chunk = (size_t)(chunk_base(tok0, b) + c) * p.H + h;
     if (tid == 0 && p0 == 0) p.decay[chunk] = expf(end);
+    if (p0 == 0) p.sums[chunk * 2 * CHUNK + tid] = tid < CHUNK ? scum[tid] : sdt[tid - CHUNK];
     {
         const bf16* xs = src + h * P + p0;
         if (vec) {
@@ -371,7 +374,9 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
     bf16* sX = sB + CHUNK * bld;                           // [CHUNK][PLD]
     bf16* sHi = sX + CHUNK * PLD;                          // [npad][PLD]: S_0
     bf16* sLo = sHi + npad * PLD;
-    __shared__ float scum[CHUNK], sdt[CHUNK];
+    __shared__ float sums[2 * CHUNK];
+    const float* scum = sums;
+    const float* sdt = sums + CHUNK;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, a4 = lane & 3;
     const int h = blockIdx.y / ptiles, p0 = (blockIdx.y - h * ptiles) * PT, b = blockIdx.z, c = blockIdx.x;
     const int N = p.N, P = p.P, g = h / (p.H / p.G), inner = p.H * P;
@@ -380,13 +385,15 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
     if (c * CHUNK >= n) return;
     const int nc = min(CHUNK, n - c * CHUNK), row0 = tok0 + c * CHUNK;
     const bf16* src = (const bf16*)p.xbc + (size_t)row0 * p.ld;
+    const size_t chunk = (size_t)(chunk_base(tok0, b) + c) * p.H + h;
+    const float my_sum = p.sums[chunk * 2 * CHUNK + tid];
     load_tile(sC, bld, src + inner + (p.G + g) * N, p.ld, nc, N, npad, vec);
     load_tile(sB, bld, src + inner + g * N, p.ld, nc, N, npad, vec);
     load_tile(sX, PLD, src + h * P + p0, p.ld, nc, min(PT, P - p0), PT, vec);
     {
-        const float* rec = p.rec + ((size_t)(chunk_base(tok0, b) + c) * p.H + h) * N * P + p0;
+        const float* rec = p.rec + chunk * N * P + p0;
         const bool vec4 = P % 4 == 0;
-        constexpr int AHEAD = 8;                           // pieces under way at a time
+        constexpr int AHEAD = 16;                          // pieces under way at a time
         for (int i0 = tid; i0 < npad * (PT / 4); i0 += AHEAD * CHUNK_THREADS) {
             float4 q[AHEAD];
 #pragma unroll
@@ -415,7 +422,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
             }
         }
     }
-    chunk_decays(p, row0, nc, h, scum, sdt);
+    sums[tid] = my_sum;
     copies_done();
     __syncthreads();
     const int t0 = warp * 16;
@@ -620,7 +627,8 @@ LLB_API int llb_ssd_scan(SsdParams p, int x_dtype, int B, cudaStream_t stream) {
     return (int)cudaErrorInvalidValue;
 }
 
-// Chunks of the step's scratch for T packed tokens of B sequences: p.rec holds chunks * H N P floats, p.decay chunks * H.
+// Chunks of the step's scratch for T packed tokens of B sequences: p.rec holds chunks * H N P floats, p.decay chunks * H, p.sums
+// chunks * H * 128.
 LLB_API int llb_ssd_chunks(int T, int B) { return T / CHUNK + B + 1; }
 
 // The same recurrence in chunks (bfloat16 operands).

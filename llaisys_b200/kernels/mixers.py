@@ -255,7 +255,8 @@ def conv_heads(x: torch.Tensor, n_q: int, n_k: int, d: int, w: torch.Tensor, sta
 class _SsdParams(ctypes.Structure):
     _fields_ = [("xbc", c_void_p), ("ld", c_int), ("dt", c_void_p), ("dt_ld", c_int), ("dt_bias", c_void_p), ("a_log", c_void_p),
                 ("skip", c_void_p), ("state", c_void_p), ("seq_start", c_void_p), ("seq_slot", c_void_p), ("out", c_void_p),
-                ("H", c_int), ("P", c_int), ("N", c_int), ("G", c_int), ("rec", c_void_p), ("decay", c_void_p)]
+                ("H", c_int), ("P", c_int), ("N", c_int), ("G", c_int), ("rec", c_void_p), ("decay", c_void_p),
+                ("sums", c_void_p)]
 
 
 SSD_MAX_STATE = 256           # rows of a head's state
@@ -291,11 +292,11 @@ def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: 
     assert xbc.dtype == torch.bfloat16
     chunks = _fn(lib, "llb_ssd_chunks", [c_int, c_int])(T, n_seqs)
     rec = torch.empty((chunks, H * N * P), dtype=torch.float32, device=xbc.device)
-    decay = torch.empty((chunks, H), dtype=torch.float32, device=xbc.device)
-    p.rec, p.decay = rec.data_ptr(), decay.data_ptr()
+    small = torch.empty((chunks * H * 129,), dtype=torch.float32, device=xbc.device)
+    p.rec, p.sums, p.decay = rec.data_ptr(), small.data_ptr(), small[chunks * H * 128:].data_ptr()
     f = _fn(lib, "llb_ssd_chunked", [_SsdParams, c_int, c_int, c_void_p])
     _check(f(p, n_seqs, max_new, _stream()), "state space (recurrence in chunks)", 3)
-    del rec, decay
+    del rec, small
     return out
 
 
