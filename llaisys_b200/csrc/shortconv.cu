@@ -33,7 +33,8 @@ __host__ __device__ constexpr int run_length(int taps) { return taps - 1 > RUN ?
 template <typename T, int U> struct alignas(sizeof(T) * U) Piece { T v[U]; };
 
 // The convolution of PIECES pieces of U neighbouring channels (columns col[i], where have[i]) over the tokens of the run that
-// starts at token at0 of the sequence; emit(t, v) gets every token's results.
+// starts at token at0 of the sequence; emit(t, v) gets every token's results
+// (with constant taps the loop over the run is unrolled, and t - at0 is a constant there).
 template <typename T, int TAPS, int PIECES, int U, typename EMIT>
 __device__ __forceinline__ void conv_run(const ShortConv& p, const int (&col)[PIECES], const bool (&have)[PIECES], int b, int tok0, int n,
                                          int at0, EMIT&& emit) {
@@ -203,15 +204,40 @@ __global__ void __launch_bounds__(THREADS) conv_heads_kernel(ConvHeads p) {
     T* kpool = (T*)p.kpool;
     T* vpool = (T*)p.vpool;
     const int pos0 = __ldg(p.tok_pos + tok0);              // (a sequence's tokens of a step stand at consecutive positions)
+    if (p.rot > 0 && (pos0 < 0 || pos0 + n > p.table_rows)) {
+        atomicExch(p.err, 2);
+        return;
+    }
+    // what the run's tokens need beside their inputs is under way before the convolution waits for those: the angles, and where
+    // the (at most two) pages of a short run's cache rows lie
+    constexpr bool AHEAD = TAPS > 0;
+    constexpr int NA = AHEAD ? RUN : 1;
+    float ca[NA][U], sa[NA][U];
+    const bool store_any = is_k && p.append;
+    size_t page_at[2] = {0, 0};
+    const int lp0 = (pos0 + at0) / LLB_PAGE;
+    if constexpr (AHEAD) {
+        if (pair)
+#pragma unroll
+            for (int u = 0; u < RUN; ++u)
+#pragma unroll
+                for (int e = 0; e < U; ++e) {
+                    const bool in = at0 + u < n;
+                    ca[u][e] = in ? __ldg(p.cos_t + (size_t)(pos0 + at0 + u) * half + first + e) : 1.f;
+                    sa[u][e] = in ? __ldg(p.sin_t + (size_t)(pos0 + at0 + u) * half + first + e) : 0.f;
+                }
+        if (store_any) {
+            const int lp1 = (pos0 + min(n, at0 + RUN) - 1) / LLB_PAGE;
+            page_at[0] = paged_row(table, p.ring, lp0 * LLB_PAGE, kvh, p.n_k, p.d, p.pinned);
+            page_at[1] = lp1 != lp0 ? paged_row(table, p.ring, lp1 * LLB_PAGE, kvh, p.n_k, p.d, p.pinned) : page_at[0];
+        }
+    }
     conv_run<T, TAPS, 2, U>(p.conv, col, have, b, tok0, n, at0, [&](int t, float (&v)[2][U]) {
         const int pos = pos0 + t;
-        if (p.rot > 0 && (pos < 0 || pos >= p.table_rows)) {
-            atomicExch(p.err, 2);
-            return;
-        }
         T* row = (T*)p.out + (size_t)(tok0 + t) * p.ldo;
-        const bool store = is_k && p.append && paged_survives(pos / LLB_PAGE, last / LLB_PAGE, p.ring, p.pinned);
-        const size_t at = store ? paged_row(table, p.ring, pos, kvh, p.n_k, p.d, p.pinned) : 0;
+        const bool store = store_any && paged_survives(pos / LLB_PAGE, last / LLB_PAGE, p.ring, p.pinned);
+        const size_t at = !store ? 0 : AHEAD ? (pos / LLB_PAGE == lp0 ? page_at[0] : page_at[1]) + (size_t)(pos % LLB_PAGE) * p.d
+                                             : paged_row(table, p.ring, pos, kvh, p.n_k, p.d, p.pinned);
         Piece<T, U> q[2];
         if (is_k) {
 #pragma unroll
@@ -226,7 +252,8 @@ __global__ void __launch_bounds__(THREADS) conv_heads_kernel(ConvHeads p) {
         if (pair) {
 #pragma unroll
             for (int e = 0; e < U; ++e) {
-                const float c = __ldg(p.cos_t + (size_t)pos * half + first + e), s = __ldg(p.sin_t + (size_t)pos * half + first + e);
+                const float c = AHEAD ? ca[t - at0][e] : __ldg(p.cos_t + (size_t)pos * half + first + e);
+                const float s = AHEAD ? sa[t - at0][e] : __ldg(p.sin_t + (size_t)pos * half + first + e);
                 const float x0 = v[0][e], x1 = v[1][e];
                 v[0][e] = x0 * c - x1 * s;
                 v[1][e] = x1 * c + x0 * s;

@@ -32,7 +32,8 @@ struct SsdParams {
     const int* seq_slot;      // [B]
     float* out;               // [T, H P]
     int H, P, N, G;
-    float* rec;               // [chunks, H, N P]: a chunk's own sum, then the state it starts with
+    float* rec;               // [chunks, H, N P]: a chunk's own sum, then the state it starts with (where rows are whole pieces
+                              // of 8: 8 leading halves and then 8 remainders, bfloat16, in the place of 8 floats)
     float* decay;             // [chunks, H]: exp(c_end)
     float* sums;              // [chunks, H, 2 * 64]: c_t of the chunk's tokens, then their steps
 };
@@ -327,7 +328,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_state_kernel(SsdParam
 // rec of every chunk: its own sum in, the state it starts with out; the sequence's state is brought up to date.
 template <int V>
 __global__ void __launch_bounds__(128) ssd_chunk_prefix_kernel(SsdParams p) {
-    constexpr int AHEAD = 8;
+    constexpr int AHEAD = V == 8 ? 4 : 8;
     const int h = blockIdx.y, b = blockIdx.z, n_el = p.N * p.P, e0 = (blockIdx.x * 128 + threadIdx.x) * V;
     llb_grid_dependency_sync();
     const int tok0 = p.seq_start[b], n = p.seq_start[b + 1] - tok0, nc = (n + CHUNK - 1) / CHUNK;
@@ -338,12 +339,27 @@ __global__ void __launch_bounds__(128) ssd_chunk_prefix_kernel(SsdParams p) {
     const float* dec = p.decay + first;
     float S[V];
     auto load = [&](float (&v)[V], const float* src) {
-        if constexpr (V == 4) { const float4 q = *reinterpret_cast<const float4*>(src); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
-        else v[0] = src[0];
+        if constexpr (V == 8) {
+            const float4 q = reinterpret_cast<const float4*>(src)[0], r = reinterpret_cast<const float4*>(src)[1];
+            v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; v[4] = r.x; v[5] = r.y; v[6] = r.z; v[7] = r.w;
+        } else v[0] = src[0];
     };
     auto store = [&](float* dst, const float (&v)[V]) {
-        if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
-        else dst[0] = v[0];
+        if constexpr (V == 8) {
+            reinterpret_cast<float4*>(dst)[0] = make_float4(v[0], v[1], v[2], v[3]);
+            reinterpret_cast<float4*>(dst)[1] = make_float4(v[4], v[5], v[6], v[7]);
+        } else dst[0] = v[0];
+    };
+    auto store_start = [&](float* dst, const float (&v)[V]) {
+        if constexpr (V == 8) {
+            uint4 hi, lo;
+            split2(v[0], v[1], hi.x, lo.x);
+            split2(v[2], v[3], hi.y, lo.y);
+            split2(v[4], v[5], hi.z, lo.z);
+            split2(v[6], v[7], hi.w, lo.w);
+            reinterpret_cast<uint4*>(dst)[0] = hi;
+            reinterpret_cast<uint4*>(dst)[1] = lo;
+        } else dst[0] = v[0];
     };
     load(S, st);
     for (int c0 = 0; c0 < nc; c0 += AHEAD) {
@@ -357,7 +373,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_prefix_kernel(SsdParams p) {
 #pragma unroll
         for (int k = 0; k < AHEAD; ++k)
             if (c0 + k < nc) {
-                store(rec + (size_t)(c0 + k) * step, S);
+                store_start(rec + (size_t)(c0 + k) * step, S);
 #pragma unroll
                 for (int e = 0; e < V; ++e) S[e] = fmaf(a[k], S[e], d[k][e]);
             }
@@ -392,33 +408,21 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
     load_tile(sX, PLD, src + h * P + p0, p.ld, nc, min(PT, P - p0), PT, vec);
     {
         const float* rec = p.rec + chunk * N * P + p0;
-        const bool vec4 = P % 4 == 0;
-        constexpr int AHEAD = 16;                          // pieces under way at a time
-        for (int i0 = tid; i0 < npad * (PT / 4); i0 += AHEAD * CHUNK_THREADS) {
-            float4 q[AHEAD];
-#pragma unroll
-            for (int k = 0; k < AHEAD; ++k) {
-                const int i = i0 + k * CHUNK_THREADS, r = i / (PT / 4), cc = (i - r * (PT / 4)) * 4;
-                q[k] = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (r >= N || p0 + cc >= P) continue;
-                const float* s = rec + (size_t)r * P + cc;
-                if (vec4) q[k] = *reinterpret_cast<const float4*>(s);
-                else {
-                    q[k].x = s[0];
-                    if (p0 + cc + 1 < P) q[k].y = s[1];
-                    if (p0 + cc + 2 < P) q[k].z = s[2];
-                    if (p0 + cc + 3 < P) q[k].w = s[3];
-                }
+        if (vec) {
+            for (int i = tid; i < npad * (PT / 8); i += CHUNK_THREADS) {
+                const int r = i / (PT / 8), cc = (i - r * (PT / 8)) * 8;
+                const bool in = r < N && p0 + cc < P;
+                const bf16* piece = reinterpret_cast<const bf16*>(in ? rec + (size_t)r * P + cc : rec);
+                copy16(sHi + r * PLD + cc, piece, in);
+                copy16(sLo + r * PLD + cc, piece + 8, in);
             }
-#pragma unroll
-            for (int k = 0; k < AHEAD; ++k) {
-                const int i = i0 + k * CHUNK_THREADS, r = i / (PT / 4), cc = (i - r * (PT / 4)) * 4;
-                if (r >= npad) break;
-                uint2 hi, lo;
-                split2(q[k].x, q[k].y, hi.x, lo.x);
-                split2(q[k].z, q[k].w, hi.y, lo.y);
-                *reinterpret_cast<uint2*>(sHi + r * PLD + cc) = hi;
-                *reinterpret_cast<uint2*>(sLo + r * PLD + cc) = lo;
+        } else {
+            for (int i = tid; i < npad * PT; i += CHUNK_THREADS) {
+                const int r = i / PT, cc = i - r * PT;
+                const float v = (r < N && p0 + cc < P) ? rec[(size_t)r * P + cc] : 0.f;
+                const bf16 hi = __float2bfloat16_rn(v);
+                sHi[r * PLD + cc] = hi;
+                sLo[r * PLD + cc] = __float2bfloat16_rn(v - __bfloat162float(hi));
             }
         }
     }
@@ -646,7 +650,7 @@ LLB_API int llb_ssd_chunked(SsdParams p, int B, int max_new, cudaStream_t stream
         llb_launch(ssd_chunk_state_kernel, dim3(chunks, p.H * ptiles, B), dim3(CHUNK_THREADS), smem, stream, p, npad, ptiles, vec);
         if (int rc = llb_status()) return rc;
     }
-    if ((p.N * p.P) % 4 == 0) llb_launch(ssd_chunk_prefix_kernel<4>, dim3((p.N * p.P / 4 + 127) / 128, p.H, B), dim3(128), 0, stream, p);
+    if (vec) llb_launch(ssd_chunk_prefix_kernel<8>, dim3((p.N * p.P / 8 + 127) / 128, p.H, B), dim3(128), 0, stream, p);
     else llb_launch(ssd_chunk_prefix_kernel<1>, dim3((p.N * p.P + 127) / 128, p.H, B), dim3(128), 0, stream, p);
     if (int rc = llb_status()) return rc;
     {

@@ -103,7 +103,7 @@ class GatedMLP(FeedForward):
 
     def forward(self, x, ctx):
         act = self._activated(x)
-        return kernels.linear(act, self.down, self.b_down, out_dtype=delta_dtype(act))
+        return kernels.linear_f32(act, self.down, self.b_down)          # (see delta_dtype)
 
     def forward_into(self, x, ctx, residual):
         if self.form is not None and kernels.mlp_fused_ok(x, self.gate_up, self.down, residual):

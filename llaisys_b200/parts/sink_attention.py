@@ -148,7 +148,7 @@ class WindowedSinkAttention(Mixer):
             self.r1, self.r2 = tensors[n["r1"]].float().contiguous(), tensors[n["r2"]].float().contiguous()
 
     def forward(self, x, ctx, call):
-        return kernels.linear(self._attend(x, ctx, call), self.w_o, out_dtype=torch.float32 if self.out_f32 else None)
+        return (kernels.linear_f32 if self.out_f32 else kernels.linear)(self._attend(x, ctx, call), self.w_o)
 
     def forward_into(self, x, ctx, call, residual):
         if not (x.dtype == torch.bfloat16 and self.w_o.dtype == torch.bfloat16

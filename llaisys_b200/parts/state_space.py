@@ -84,7 +84,7 @@ class StateSpace(Mixer):
         return kernels.gated_group_norm(y, proj[:, :self.inner], self.w_norm, self.norm_groups, self.eps, x.dtype)
 
     def forward(self, x, ctx, call):
-        return kernels.linear(self._heads(x, ctx, call), self.w_o, out_dtype=torch.float32)
+        return kernels.linear_f32(self._heads(x, ctx, call), self.w_o)
 
     def forward_into(self, x, ctx, call, residual):
         if not (x.dtype == torch.bfloat16 and self.w_o.dtype == torch.bfloat16
