@@ -179,17 +179,19 @@ __device__ __forceinline__ void copies_done() { asm volatile("cp.async.wait_all;
 
 // [CHUNK rows, cols] of the operand into a tile of `pad` columns (a multiple of 16): 16-byte asynchronous copies where the rows
 // allow it; zeros beyond `cols` and beyond the chunk's tokens.
+template <int THREADS>
 __device__ __forceinline__ void load_tile(bf16* dst, int dst_ld, const bf16* src, int ld, int rows, int cols, int pad, bool vec) {
     const int tid = threadIdx.x;
-    if (vec) {
-        const int per = pad / 8;
-        for (int i = tid; i < CHUNK * per; i += CHUNK_THREADS) {
-            const int r = i / per, c = (i - r * per) * 8;
-            const bool in = r < rows && c < cols;
-            copy16(dst + r * dst_ld + c, in ? src + (size_t)r * ld + c : src, in);
+    if (vec) {                                             // 16 threads a row
+        const int sub = (tid & 15) * 8;
+#pragma unroll
+        for (int k = 0; k < CHUNK * 16 / THREADS; ++k) {
+            const int r = (tid >> 4) + k * (THREADS / 16);
+            const bf16* row = src + (size_t)r * ld;
+            for (int c = sub; c < pad; c += 128) copy16(dst + r * dst_ld + c, r < rows && c < cols ? row + c : src, r < rows && c < cols);
         }
     } else {
-        for (int i = tid; i < CHUNK * pad; i += CHUNK_THREADS) {
+        for (int i = tid; i < CHUNK * pad; i += THREADS) {
             const int r = i / pad, c = i - r * pad;
             dst[r * dst_ld + c] = (r < rows && c < cols) ? src[(size_t)r * ld + c] : __float2bfloat16_rn(0.f);
         }
@@ -238,7 +240,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_state_kernel(SsdParam
     if (c * CHUNK >= n) return;
     const int nc = min(CHUNK, n - c * CHUNK), row0 = tok0 + c * CHUNK;
     const bf16* src = (const bf16*)p.xbc + (size_t)row0 * p.ld;
-    load_tile(sB, bld, src + inner + g * N, p.ld, nc, N, npad, vec);
+    load_tile<CHUNK_THREADS>(sB, bld, src + inner + g * N, p.ld, nc, N, npad, vec);
     // (the rows of x are under way before the decays are formed)
     constexpr int XP = CHUNK * (PT / 8) / CHUNK_THREADS;
     uint4 xq[XP];
@@ -288,40 +290,53 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_state_kernel(SsdParam
     const uint32_t ab = smem_addr(sB) + (((lane & 7) + ((lane >> 4) << 3)) * bld + ((lane >> 3) & 1) * 8) * 2;
     const uint32_t xoff = ((lane & 15) * PLD + (lane >> 4) * 8) * 2;
     const uint32_t hb = smem_addr(sHi) + xoff, lb = smem_addr(sLo) + xoff;
-    for (int m0 = warp * 16; m0 < npad; m0 += CHUNK_THREADS / 32 * 16) {
-        float acc[PT / 8][4];
+    constexpr int MSTEP = CHUNK_THREADS / 32 * 16;         // a warp takes two tiles of 16 rows, this far apart, for every tile of x it loads
+    for (int m0 = warp * 16; m0 < npad; m0 += 2 * MSTEP) {
+        const bool two = m0 + MSTEP < npad;
+        float acc[2][PT / 8][4];
 #pragma unroll
-        for (int j = 0; j < PT / 8; ++j)
+        for (int m = 0; m < 2; ++m)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
+            for (int j = 0; j < PT / 8; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc[m][j][e] = 0.f;
 #pragma unroll
         for (int k0 = 0; k0 < CHUNK; k0 += 16) {
-            uint32_t a[4];
-            ldsm_t(a, ab + (k0 * bld + m0) * 2);
+            uint32_t a[2][4];
+            ldsm_t(a[0], ab + (k0 * bld + m0) * 2);
+            if (two) ldsm_t(a[1], ab + (k0 * bld + m0 + MSTEP) * 2);
 #pragma unroll
             for (int j = 0; j < PT / 16; ++j) {
-                uint32_t x[4];
+                uint32_t x[4], y[4];
                 ldsm_t(x, hb + (k0 * PLD + j * 16) * 2);
-                mma(acc[2 * j], a, x[0], x[1]);
-                mma(acc[2 * j + 1], a, x[2], x[3]);
-                ldsm_t(x, lb + (k0 * PLD + j * 16) * 2);
-                mma(acc[2 * j], a, x[0], x[1]);
-                mma(acc[2 * j + 1], a, x[2], x[3]);
+                ldsm_t(y, lb + (k0 * PLD + j * 16) * 2);
+#pragma unroll
+                for (int m = 0; m < 2; ++m) {
+                    if (m && !two) break;
+                    mma(acc[m][2 * j], a[m], x[0], x[1]);
+                    mma(acc[m][2 * j + 1], a[m], x[2], x[3]);
+                    mma(acc[m][2 * j], a[m], y[0], y[1]);
+                    mma(acc[m][2 * j + 1], a[m], y[2], y[3]);
+                }
             }
         }
 #pragma unroll
-        for (int j = 0; j < PT / 8; ++j)
+        for (int m = 0; m < 2; ++m) {
+            if (m && !two) break;
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int i = m0 + g8 + half * 8, cc = p0 + j * 8 + a4 * 2;
-                if (i >= N || cc >= P) continue;
-                float* dst = rec + (size_t)i * P + cc;
-                if (P % 2 == 0) *reinterpret_cast<float2*>(dst) = make_float2(acc[j][half * 2], acc[j][half * 2 + 1]);
-                else {
-                    dst[0] = acc[j][half * 2];
-                    if (cc + 1 < P) dst[1] = acc[j][half * 2 + 1];
+            for (int j = 0; j < PT / 8; ++j)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const int i = m0 + m * MSTEP + g8 + half * 8, cc = p0 + j * 8 + a4 * 2;
+                    if (i >= N || cc >= P) continue;
+                    float* dst = rec + (size_t)i * P + cc;
+                    if (P % 2 == 0) *reinterpret_cast<float2*>(dst) = make_float2(acc[m][j][half * 2], acc[m][j][half * 2 + 1]);
+                    else {
+                        dst[0] = acc[m][j][half * 2];
+                        if (cc + 1 < P) dst[1] = acc[m][j][half * 2 + 1];
+                    }
                 }
-            }
+        }
     }
 }
 
@@ -381,8 +396,10 @@ __global__ void __launch_bounds__(128) ssd_chunk_prefix_kernel(SsdParams p) {
     store(st, S);
 }
 
-// y of one chunk of one head, PT columns: a warp takes 16 tokens.
-__global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams p, int npad, int ptiles, int vec) {
+// y of one chunk of one head, PT columns: a warp takes 16 tokens and half of the columns (both halves' warps form the scores: that
+// costs a quarter more products and doubles the warps that an SM's shared memory has room for).
+constexpr int OUT_THREADS = 256, OUT_COLS = PT / 2;
+__global__ void __launch_bounds__(OUT_THREADS) ssd_chunk_out_kernel(SsdParams p, int npad, int ptiles, int vec) {
     extern __shared__ __align__(16) unsigned char raw[];
     const int bld = npad + 8;
     bf16* sC = reinterpret_cast<bf16*>(raw);               // [CHUNK][bld]
@@ -402,14 +419,14 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
     const int nc = min(CHUNK, n - c * CHUNK), row0 = tok0 + c * CHUNK;
     const bf16* src = (const bf16*)p.xbc + (size_t)row0 * p.ld;
     const size_t chunk = (size_t)(chunk_base(tok0, b) + c) * p.H + h;
-    const float my_sum = p.sums[chunk * 2 * CHUNK + tid];
-    load_tile(sC, bld, src + inner + (p.G + g) * N, p.ld, nc, N, npad, vec);
-    load_tile(sB, bld, src + inner + g * N, p.ld, nc, N, npad, vec);
-    load_tile(sX, PLD, src + h * P + p0, p.ld, nc, min(PT, P - p0), PT, vec);
+    const float my_sum = tid < 2 * CHUNK ? p.sums[chunk * 2 * CHUNK + tid] : 0.f;
+    load_tile<OUT_THREADS>(sC, bld, src + inner + (p.G + g) * N, p.ld, nc, N, npad, vec);
+    load_tile<OUT_THREADS>(sB, bld, src + inner + g * N, p.ld, nc, N, npad, vec);
+    load_tile<OUT_THREADS>(sX, PLD, src + h * P + p0, p.ld, nc, min(PT, P - p0), PT, vec);
     {
         const float* rec = p.rec + chunk * N * P + p0;
         if (vec) {
-            for (int i = tid; i < npad * (PT / 8); i += CHUNK_THREADS) {
+            for (int i = tid; i < npad * (PT / 8); i += OUT_THREADS) {
                 const int r = i / (PT / 8), cc = (i - r * (PT / 8)) * 8;
                 const bool in = r < N && p0 + cc < P;
                 const bf16* piece = reinterpret_cast<const bf16*>(in ? rec + (size_t)r * P + cc : rec);
@@ -417,7 +434,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
                 copy16(sLo + r * PLD + cc, piece + 8, in);
             }
         } else {
-            for (int i = tid; i < npad * PT; i += CHUNK_THREADS) {
+            for (int i = tid; i < npad * PT; i += OUT_THREADS) {
                 const int r = i / PT, cc = i - r * PT;
                 const float v = (r < N && p0 + cc < P) ? rec[(size_t)r * P + cc] : 0.f;
                 const bf16 hi = __float2bfloat16_rn(v);
@@ -426,18 +443,18 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
             }
         }
     }
-    sums[tid] = my_sum;
+    if (tid < 2 * CHUNK) sums[tid] = my_sum;
     copies_done();
     __syncthreads();
-    const int t0 = warp * 16;
-    if (t0 >= nc) return;                                  // (no barrier follows)
+    const int t0 = (warp & 3) * 16, col0 = (warp >> 2) * OUT_COLS;
+    if (t0 >= nc || p0 + col0 >= P) return;                // (no barrier follows)
     const uint32_t ca = smem_addr(sC) + ((t0 + (lane & 15)) * bld + (lane >> 4) * 8) * 2;
     const uint32_t bb = smem_addr(sB) + (((lane & 7) + ((lane >> 4) << 3)) * bld + ((lane >> 3) & 1) * 8) * 2;
-    const uint32_t xoff = ((lane & 15) * PLD + (lane >> 4) * 8) * 2;
+    const uint32_t xoff = ((lane & 15) * PLD + (lane >> 4) * 8 + col0) * 2;
     const uint32_t xb = smem_addr(sX) + xoff, hb = smem_addr(sHi) + xoff, lb = smem_addr(sLo) + xoff;
-    float acc[PT / 8][4];
+    float acc[OUT_COLS / 8][4];
 #pragma unroll
-    for (int j = 0; j < PT / 8; ++j)
+    for (int j = 0; j < OUT_COLS / 8; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
     // ---- what the chunk starts with
@@ -446,7 +463,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
         uint32_t a[4];
         ldsm(a, ca + k0 * 2);
 #pragma unroll
-        for (int j = 0; j < PT / 16; ++j) {
+        for (int j = 0; j < OUT_COLS / 16; ++j) {
             uint32_t s[4];
             ldsm_t(s, hb + (k0 * PLD + j * 16) * 2);
             mma(acc[2 * j], a, s[0], s[1]);
@@ -459,7 +476,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
     const float ct[2] = {scum[t0 + g8], scum[t0 + g8 + 8]};
     const float et[2] = {expf(ct[0]), expf(ct[1])};
 #pragma unroll
-    for (int j = 0; j < PT / 8; ++j)
+    for (int j = 0; j < OUT_COLS / 8; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[j][e] *= et[e >> 1];
     // ---- the chunk's own tokens, 16 at a time
@@ -490,7 +507,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
         split2(w[1][0], w[1][1], hi[2], lo[2]);
         split2(w[1][2], w[1][3], hi[3], lo[3]);
 #pragma unroll
-        for (int j = 0; j < PT / 16; ++j) {
+        for (int j = 0; j < OUT_COLS / 16; ++j) {
             uint32_t x[4];
             ldsm_t(x, xb + (s0 * PLD + j * 16) * 2);
             mma(acc[2 * j], hi, x[0], x[1]);
@@ -501,10 +518,10 @@ __global__ void __launch_bounds__(CHUNK_THREADS) ssd_chunk_out_kernel(SsdParams 
     }
     const float skip = p.skip[h];
 #pragma unroll
-    for (int j = 0; j < PT / 8; ++j)
+    for (int j = 0; j < OUT_COLS / 8; ++j)
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-            const int t = t0 + g8 + half * 8, cl = j * 8 + a4 * 2, cc = p0 + cl;
+            const int t = t0 + g8 + half * 8, cl = col0 + j * 8 + a4 * 2, cc = p0 + cl;
             if (t >= nc || cc >= P) continue;
             float* dst = p.out + (size_t)(row0 + t) * inner + h * P + cc;
             const float y0 = fmaf(skip, __bfloat162float(sX[t * PLD + cl]), acc[j][half * 2]);
@@ -657,7 +674,7 @@ LLB_API int llb_ssd_chunked(SsdParams p, int B, int max_new, cudaStream_t stream
         static int have = 0;
         const size_t smem = 2 * tile + xt + 2 * (size_t)npad * PLD * 2;
         if (int rc = set_smem((const void*)ssd_chunk_out_kernel, have, smem)) return rc;
-        llb_launch(ssd_chunk_out_kernel, dim3(chunks, p.H * ptiles, B), dim3(CHUNK_THREADS), smem, stream, p, npad, ptiles, vec);
+        llb_launch(ssd_chunk_out_kernel, dim3(chunks, p.H * ptiles, B), dim3(OUT_THREADS), smem, stream, p, npad, ptiles, vec);
     }
     return llb_status();
 }
